@@ -74,3 +74,7 @@ def _register_builtin() -> None:
     from . import tinevik as _tvc
     register_architecture(Architecture(_tvc.ARCHITECTURE, _tvc.TinevikConfig.from_dict, _tv.tinevik_manifest, _tv.build_tinevik,
                                        _tv.is_norm_weight), replace=True)
+    from ..models import lirutar as _lr
+    from . import lirutar as _lrc
+    register_architecture(Architecture(_lrc.ARCHITECTURE, _lrc.LirutarConfig.from_dict, _lr.lirutar_manifest, _lr.build_lirutar,
+                                       _lr.is_norm_weight), replace=True)

@@ -46,7 +46,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 2) attention_decode_kernel(
     const int32_t* __restrict__ token_seg, const int32_t* __restrict__ positions, const int32_t* __restrict__ tok_list,
     T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int nh, int nkv,
     int hd, int page_size, int max_blocks, int max_splits, float scale, int window, int vd, const float* __restrict__ dist_bias,
-    int max_dist, int v_in_key, int v_share) {
+    int max_dist, int v_in_key, int v_share, int out_ld) {
     constexpr int V = Vec16<T>::N;
     extern __shared__ float smem[];
     const int g = nh / nkv;
@@ -248,7 +248,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 2) attention_decode_kernel(
         for (int d = tid; d < vd; d += DEC_THREADS) {
             float o = 0.0f;
             for (int gi = 0; gi < parts; gi++) o += red[gi * vd + d];
-            if (single) out[((size_t)t * nh + h0 + h) * vd + d] = from_f32<T>(o * (1.0f / stat_l[h]));
+            if (single) out[(size_t)t * out_ld + (size_t)(h0 + h) * vd + d] = from_f32<T>(o * (1.0f / stat_l[h]));
             else part_o[(((size_t)zi * nh + h0 + h) * max_splits + split) * vd + d] = o;
         }
     }
@@ -307,7 +307,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 2) attention_decode_kernel(
             o += a3 * wsp[h * DEC_SPLIT + j + 3];
         }
         for (; j < n_active; j++) o += __ldcg(po + (size_t)j * vd) * wsp[h * DEC_SPLIT + j];
-        out[((size_t)t * nh + h0 + h) * vd + d] = from_f32<T>(o * stat_l[h]);
+        out[(size_t)t * out_ld + (size_t)(h0 + h) * vd + d] = from_f32<T>(o * stat_l[h]);
     }
 }
 
@@ -384,7 +384,7 @@ VK_API int vk_attention_decode(const void* q, const void* cache, const int32_t* 
         }                                                                                                                            \
         return launch_dependent(kern, grid, dim3(DEC_THREADS), smem, stream, (const T*)q, (const T*)cache, block_tables, token_seg, \
                                 positions, tok_list, (T*)out, part_o, part_ml, counters, nh, nkv, hd, page_size, max_blocks, splits, \
-                                scale, window, hd, (const float*)nullptr, 0, 0, 1);                                                  \
+                                scale, window, hd, (const float*)nullptr, 0, 0, 1, nh * hd);                                         \
     }
     if (dtype == 0) {
         if (async) GO(float, true) else GO(float, false)
@@ -397,15 +397,16 @@ VK_API int vk_attention_decode(const void* q, const void* cache, const int32_t* 
 
 // The same for the unrotated form of the attention: values of size vd (the scratch is
 // vk_attention_decode_scratch_bytes(tokens, nh, nkv, max(hd, vd), max_context) bytes) and an optional bias by distance.
-// v_in_key: the cache holds keys alone and a key's first vd values are its value (vd <= hd).
+// v_in_key: the cache holds keys alone and a key's first vd values are its value (vd <= hd).  Rows of out are out_ld elements apart.
 // v_share > 1: key heads v_share*j .. v_share*j + v_share-1 read value head j (a page holds nkv / v_share heads of values).
 // Always the CUDA-core kernel, in both dtypes.
 VK_API int vk_attention_decode_biased(const void* q, const void* cache, const int32_t* block_tables, const int32_t* token_seg,
                                       const int32_t* positions, const int32_t* tok_list, void* out, void* scratch, int scratch_tokens,
                                       int n_tokens, int nh, int nkv, int hd, int vd, int page_size, int max_blocks, int max_context,
                                       int grid_context, float scale, int window, const float* dist_bias, int max_dist, int v_in_key,
-                                      int v_share, int dtype, cudaStream_t stream) {
+                                      int v_share, int out_ld, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return VK_OK;
+    if (out_ld < nh * vd) return VK_BAD_SHAPE;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || hd <= 0 || vd <= 0 || page_size <= 0 || max_blocks <= 0 || window < 0 || max_context <= 0 ||
         grid_context <= 0 || grid_context > max_context || (dist_bias && max_dist <= 0))
         return VK_BAD_SHAPE;
@@ -438,7 +439,7 @@ VK_API int vk_attention_decode_biased(const void* q, const void* cache, const in
         }                                                                                                                            \
         return launch_dependent(kern, grid, dim3(DEC_THREADS), smem, stream, (const T*)q, (const T*)cache, block_tables, token_seg, \
                                 positions, tok_list, (T*)out, part_o, part_ml, counters, nh, nkv, hd, page_size, max_blocks, splits, \
-                                scale, window, vd, dist_bias, max_dist, v_in_key, v_share);                                          \
+                                scale, window, vd, dist_bias, max_dist, v_in_key, v_share, out_ld);                                  \
     }
     if (dtype == 0) {
         if (async) GO(float, true) else GO(float, false)
@@ -517,7 +518,7 @@ VK_API int vk_attention_decode_static(const void* q, const void* cache, const in
         }                                                                                                                     \
         kern<<<grid, DEC_THREADS, smem, stream>>>((const T*)q, (const T*)cache, block_tables, token_seg, positions, tok_list, \
                                                   (T*)out, part_o, part_ml, counters, nh, nkv, hd, page_size, max_blocks,     \
-                                                  splits, scale, window, hd, (const float*)nullptr, 0, 0, 1);                 \
+                                                  splits, scale, window, hd, (const float*)nullptr, 0, 0, 1, nh * hd);        \
     }
     if (dtype == 0) {
         if (async) GO(float, true) else GO(float, false)

@@ -7,8 +7,9 @@
 //  p_h(i, .)      = softmax of z'_h over the keys j <= i (inside the window, if there is one)
 //  o_h(i)         = sum_j p_h(i, j) v_j, turned back by -i * g_m
 //
-//  mixed_attn_prepare   one block a token, a warp a head: from the float32 row of the first product [ q | k | v ] to q in the compute
-//                       dtype and k, v in the token's cache slot.
+//  mixed_attn_prepare   one block a token, a warp a head: from the float32 row of the first product [ q | k | v ] (plus a bias over its
+//                       columns, if there is one) to q in the compute dtype and k, v (times v_mult) in the token's cache slot.  The
+//                       token's cos and sin are worked out once for all heads.
 //  attention_mixed_rows one block a query token, all heads: keys in runs of 128 at absolute positions (a thread a key for the scores,
 //                       a warp a head for the softmax's running maximum and sum, a thread some (head, value) pairs for the
 //                       weighted sum), so the order of an output's sums depends on its own position alone.  Any sizes, both storage
@@ -28,7 +29,9 @@ __global__ void __launch_bounds__(256) mixed_attn_prepare_kernel(const float* __
                                                                  const int32_t* __restrict__ slot, const float* __restrict__ qn_w,
                                                                  const float* __restrict__ kn_w, float eps, const float* __restrict__ freq, int dims,
                                                                  const float* __restrict__ vfreq, T* __restrict__ q_out, T* __restrict__ cache,
-                                                                 int nh, int nkv, int hd, int vd, int page_size) {
+                                                                 int nh, int nkv, int hd, int vd, int page_size, const float* __restrict__ bias,
+                                                                 float v_mult) {
+    extern __shared__ float mp_turn[];                  // cos and sin of the token's angles: [dims/2][2] for q and k, then [vd/2][2] for v
     dependency_wait();
     let_dependents_start();
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -40,42 +43,50 @@ __global__ void __launch_bounds__(256) mixed_attn_prepare_kernel(const float* __
     const int off = s >= 0 ? s % page_size : 0;
     const float pos = (float)positions[t];
     const int half = dims / 2, vhalf = vd / 2;
+    for (int i = threadIdx.x; i < half + (vfreq ? vhalf : 0); i += blockDim.x) {
+        const float ang = pos * (i < half ? freq[i] : vfreq[i - half]);
+        mp_turn[2 * i] = cosf(ang);
+        mp_turn[2 * i + 1] = sinf(ang);
+    }
+    __syncthreads();
     for (int h = warp; h < nh + 2 * nkv; h += nwarps) {
         if (h < nh + nkv) {                             // a query or key head: norm, weight, rotation
             const float* v = in + (size_t)h * hd;
             const float* w = h < nh ? qn_w : kn_w;
             T* dst = h < nh ? q_out + ((size_t)t * nh + h) * hd : (s >= 0 ? kbase + ((size_t)(h - nh) * page_size + off) * hd : nullptr);
             if (!dst) continue;
+            const float* bh = bias ? bias + (size_t)h * hd : nullptr;
+            auto at = [&](int d) { return bh ? v[d] + bh[d] : v[d]; };
             float inv = 1.0f;
             if (eps >= 0.0f) {
                 float ss = 0.0f;
-                for (int d = lane; d < hd; d += 32) ss = fmaf(v[d], v[d], ss);
+                for (int d = lane; d < hd; d += 32) { const float e = at(d); ss = fmaf(e, e, ss); }
                 ss = warp_sum(ss);
                 inv = 1.0f / sqrtf(ss / (float)hd + eps);
             }
             for (int i = lane; i < half; i += 32) {
-                const float ang = pos * freq[i];
-                const float c = cosf(ang), sn = sinf(ang);
-                const float a = (v[i] * inv) * (w ? w[i] : 1.0f), b = (v[i + half] * inv) * (w ? w[i + half] : 1.0f);
+                const float c = mp_turn[2 * i], sn = mp_turn[2 * i + 1];
+                const float a = (at(i) * inv) * (w ? w[i] : 1.0f), b = (at(i + half) * inv) * (w ? w[i + half] : 1.0f);
                 dst[i] = from_f32<T>(a * c - b * sn);
                 dst[i + half] = from_f32<T>(b * c + a * sn);
             }
-            for (int d = dims + lane; d < hd; d += 32) dst[d] = from_f32<T>((v[d] * inv) * (w ? w[d] : 1.0f));
+            for (int d = dims + lane; d < hd; d += 32) dst[d] = from_f32<T>((at(d) * inv) * (w ? w[d] : 1.0f));
         } else if (s >= 0) {                            // a value head
             const int g = h - nh - nkv;
             const float* v = in + (size_t)(nh + nkv) * hd + (size_t)g * vd;
+            const float* bh = bias ? bias + (size_t)(nh + nkv) * hd + (size_t)g * vd : nullptr;
+            auto at = [&](int d) { return (bh ? v[d] + bh[d] : v[d]) * v_mult; };
             T* dst = vbase + ((size_t)g * page_size + off) * vd;
             if (vfreq) {
                 for (int i = lane; i < vhalf; i += 32) {
-                    const float ang = pos * vfreq[i];
-                    const float c = cosf(ang), sn = sinf(ang);
-                    const float a = v[i], b = v[i + vhalf];
+                    const float c = mp_turn[2 * (half + i)], sn = mp_turn[2 * (half + i) + 1];
+                    const float a = at(i), b = at(i + vhalf);
                     dst[i] = from_f32<T>(a * c - b * sn);
                     dst[i + vhalf] = from_f32<T>(b * c + a * sn);
                 }
-                if (vd & 1) { if (lane == 0) dst[vd - 1] = from_f32<T>(v[vd - 1]); }
+                if (vd & 1) { if (lane == 0) dst[vd - 1] = from_f32<T>(at(vd - 1)); }
             } else {
-                for (int d = lane; d < vd; d += 32) dst[d] = from_f32<T>(v[d]);
+                for (int d = lane; d < vd; d += 32) dst[d] = from_f32<T>(at(d));
             }
         }
     }
@@ -601,16 +612,18 @@ using namespace vk;
 // write); qn_w, kn_w float32 [hd] or null; eps < 0: no norm; freq float32 [dims/2] (dims 0: no rotation); vfreq float32 [vd/2] or null.
 VK_API int vk_mixed_attn_prepare(const float* proj, int N, const int32_t* positions, const int32_t* slot, const float* qn_w, const float* kn_w, float eps,
                                  const float* freq, int dims, const float* vfreq, void* q_out, void* cache, int tokens, int nh, int nkv, int hd, int vd,
-                                 int page_size, int dtype, cudaStream_t stream) {
+                                 int page_size, const float* bias, float v_mult, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     if (nh <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || N < (nh + nkv) * hd + nkv * vd || dims < 0 || dims % 2 || dims > hd ||
         (dims > 0 && !freq))
         return VK_BAD_SHAPE;
+    const size_t smem = (size_t)(dims + vd + 1) * sizeof(float);
+    if (smem > 48 * 1024) return VK_TOO_LARGE;
     if (dtype == 0)
-        return launch_dependent(mixed_attn_prepare_kernel<float>, dim3(tokens), dim3(256), 0, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq, dims,
-                                vfreq, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size);
-    return launch_dependent(mixed_attn_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
-                            dims, vfreq, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size);
+        return launch_dependent(mixed_attn_prepare_kernel<float>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
+                                dims, vfreq, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);
+    return launch_dependent(mixed_attn_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
+                            dims, vfreq, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);
 }
 
 VK_API size_t vk_attention_mixed_rows_smem(int nh, int hd, int vd) {

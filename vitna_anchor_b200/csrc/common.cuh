@@ -95,6 +95,12 @@ __device__ __forceinline__ float activate_rt(int kind, float z) {
     return z;
 }
 
+// The same for the products' epilogues without a gate, which also take 4: relu squared.
+__device__ __forceinline__ float activate_dense(int kind, float z) {
+    if (kind == 4) { const float r = fmaxf(z, 0.0f); return r * r; }
+    return activate_rt(kind, z);
+}
+
 inline int launch_status() { return (int)cudaGetLastError(); }
 
 // Programmatic dependent launch.  A kernel launched with launch_dependent() may start while the kernel before it

@@ -2,6 +2,10 @@
 //
 //  experts_route     one block a token: logits z = W_r x + b in float32 (a warp a logit), the `top` largest (of equal logits the lower
 //                    index), weights = softmax over the chosen logits alone.  Writes ids [tokens][top] and weights [tokens][top].
+//  experts_route_scored  scores s = softmax(W_r x) over experts AND identities; a token's choice goes by s + correction: of `count` equal
+//                    groups of neighbours only the `keep` with the largest choice score take part, and of their members the `top` with the
+//                    largest (of equals the lower index); weights s / (sum of the chosen s + 1e-20) times scale.  An id of E or more
+//                    is an identity: its output is the token's input row.
 //  experts_route_table  ids[token][k] = table[token id][k], every weight 1 / top: the experts of a token are a function of its id.
 //  experts_gate_up   act[token, k] = f(W_gate,e x) * (W_up,e x) for the token's k-th expert e; a warp an output column, the token's row
 //                    in shared memory.  f is one of the epilogues' activations.
@@ -73,6 +77,90 @@ __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict_
     }
 }
 
+// A block TB tokens (a row of the router is read once for all of them); a warp a logit, then a warp a token.  all = experts + identities.
+template <typename T, int TB>
+__global__ void __launch_bounds__(128) experts_route_scored_kernel(const T* __restrict__ x, int width, const float* __restrict__ wr,
+                                                                   const float* __restrict__ correction, int all, int top, int count, int keep, float scale,
+                                                                   int32_t* __restrict__ ids, float* __restrict__ wts, int tokens) {
+    extern __shared__ float rs_sm[];                    // [TB][all] scores | [TB][all] choice scores | [TB][count] the groups' best
+    dependency_wait();
+    let_dependents_start();
+    const int t0 = blockIdx.x * TB, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    for (int e = warp; e < all; e += nwarps) {
+        const float* w = wr + (size_t)e * width;
+        float acc[TB];
+#pragma unroll
+        for (int b = 0; b < TB; b++) acc[b] = 0.0f;
+        for (int i = lane; i < width; i += 32) {
+            const float wv = w[i];
+#pragma unroll
+            for (int b = 0; b < TB; b++) acc[b] = fmaf(to_f32<T>(x[(size_t)min(t0 + b, tokens - 1) * width + i]), wv, acc[b]);
+        }
+#pragma unroll
+        for (int b = 0; b < TB; b++) {
+            acc[b] = warp_sum(acc[b]);
+            if (lane == 0) rs_sm[b * all + e] = acc[b];
+        }
+    }
+    __syncthreads();
+    const int t = t0 + warp;
+    if (warp >= TB || t >= tokens) return;
+    float* s = rs_sm + warp * all;
+    float* choice = rs_sm + TB * all + warp * all;
+    float* best_of = rs_sm + 2 * TB * all + warp * count;
+    float mx = -INFINITY, sum = 0.0f;
+    for (int e = lane; e < all; e += 32) mx = fmaxf(mx, s[e]);
+    mx = warp_max(mx);
+    for (int e = lane; e < all; e += 32) { const float v = expf(s[e] - mx); s[e] = v; sum += v; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < all; e += 32) {
+        const float v = s[e] / sum;
+        s[e] = v;
+        choice[e] = v + (correction ? correction[e] : 0.0f);
+    }
+    __syncwarp();
+    // the largest of n values (of equals the first), which then counts no more; every lane gets its index
+    auto take = [&](float* v, int n) {
+        float best = -INFINITY;
+        int arg = 0x7fffffff;
+        for (int i = lane; i < n; i += 32)
+            if (v[i] > best) { best = v[i]; arg = i; }
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+            if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+        }
+        if (arg >= n) arg = 0;                          // scores that are not numbers: stay inside the tables
+        if (lane == 0) v[arg] = -INFINITY;
+        __syncwarp();
+        return arg;
+    };
+    if (keep < count) {
+        const int size = all / count;
+        for (int g = lane; g < count; g += 32) {
+            float m = -INFINITY;
+            for (int i = 0; i < size; i++) m = fmaxf(m, choice[g * size + i]);
+            best_of[g] = m;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; k++) take(best_of, count);
+        for (int e = lane; e < all; e += 32)
+            if (best_of[e / size] != -INFINITY) choice[e] = -INFINITY;      // a group that was not taken
+        __syncwarp();
+    }
+    float mine = 0.0f, chosen = 0.0f;
+    int id = 0;
+    for (int k = 0; k < top; k++) {
+        const int e = take(choice, all);
+        chosen += s[e];
+        if (lane == k) { mine = s[e]; id = e; }
+    }
+    if (lane < top) {
+        ids[(size_t)t * top + lane] = id;
+        wts[(size_t)t * top + lane] = mine / (chosen + 1e-20f) * scale;
+    }
+}
+
 __global__ void __launch_bounds__(256) experts_route_table_kernel(const int32_t* __restrict__ tokens, const int32_t* __restrict__ table, int vocab,
                                                                   int table_top, int E, int top, int32_t* __restrict__ ids, float* __restrict__ wts, int n) {
     dependency_wait();
@@ -90,16 +178,17 @@ __global__ void __launch_bounds__(256) experts_route_table_kernel(const int32_t*
 // grid (pairs, column groups); a warp a column
 template <typename T>
 __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restrict__ x, int width, const T* __restrict__ wgu, int ff, int top,
-                                                              const int32_t* __restrict__ ids, int act, float limit, float alpha,
+                                                              const int32_t* __restrict__ ids, int E, int act, float limit, float alpha,
                                                               T* __restrict__ out) {
     extern __shared__ float xs[];                       // [width]
     dependency_wait();
     let_dependents_start();
     const int p = blockIdx.x, t = p / top;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const int e = ids[p];
+    if (e >= E) return;                                 // an identity
     for (int i = threadIdx.x; i < width; i += blockDim.x) xs[i] = to_f32<T>(x[(size_t)t * width + i]);
     __syncthreads();
-    const int e = ids[p];
     const T* wg = wgu + (size_t)e * 2 * ff * width;
     const T* wu = wg + (size_t)ff * width;
     for (int c = blockIdx.y * nwarps + warp; c < ff; c += gridDim.y * nwarps) {
@@ -128,7 +217,8 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
 // grid (tokens, column groups); a warp a column of y
 template <typename T>
 __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__ act, int ff, const T* __restrict__ wd, int width, int top,
-                                                           const int32_t* __restrict__ ids, const float* __restrict__ wts, float* __restrict__ y) {
+                                                           const int32_t* __restrict__ ids, const float* __restrict__ wts, float* __restrict__ y, int E,
+                                                           const T* __restrict__ x) {
     extern __shared__ float as[];                       // [top][ff]
     dependency_wait();
     let_dependents_start();
@@ -140,6 +230,10 @@ __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__
         float total = 0.0f;
         for (int k = 0; k < top; k++) {
             const int e = ids[(size_t)t * top + k];
+            if (e >= E) {                               // an identity: the input itself
+                total = fmaf(wts[(size_t)t * top + k], to_f32<T>(x[(size_t)t * width + c]), total);
+                continue;
+            }
             const T* w = wd + ((size_t)e * width + c) * ff;
             const float* a = as + (size_t)k * ff;
             float acc = 0.0f;
@@ -209,8 +303,10 @@ __global__ void __launch_bounds__(128) experts_gather_kernel(const T* __restrict
     }
 }
 
+template <typename T>
 __global__ void __launch_bounds__(256) experts_combine_kernel(const float* __restrict__ o, int width, int top, const int32_t* __restrict__ pos,
-                                                              const float* __restrict__ wts, float* __restrict__ y) {
+                                                              const float* __restrict__ wts, float* __restrict__ y, int E,
+                                                              const int32_t* __restrict__ ids, const T* __restrict__ x) {
     dependency_wait();
     let_dependents_start();
     const int t = blockIdx.x;
@@ -219,6 +315,7 @@ __global__ void __launch_bounds__(256) experts_combine_kernel(const float* __res
         for (int k = 0; k < top; k++) {
             const int r = pos[(size_t)t * top + k];
             if (r >= 0) total = fmaf(wts[(size_t)t * top + k], o[(size_t)r * width + c], total);
+            else if (ids[(size_t)t * top + k] >= E) total = fmaf(wts[(size_t)t * top + k], to_f32<T>(x[(size_t)t * width + c]), total);
         }
         y[(size_t)t * width + c] += total;
     }
@@ -254,11 +351,37 @@ VK_API int vk_experts_gather(const void* x, int width, const int32_t* row_token,
                             (__nv_bfloat16*)xs);
 }
 
-// y float32 [tokens][width] += sum_k wts[t][k] o[pos[t][k]]; o float32 [rows][width].
-VK_API int vk_experts_combine(const float* o, int width, int top, const int32_t* pos, const float* wts, float* y, int tokens, cudaStream_t stream) {
+// y float32 [tokens][width] += sum_k wts[t][k] o[pos[t][k]]; o float32 [rows][width]; ids of E and more: the token's row of x [tokens][width].
+VK_API int vk_experts_combine(const float* o, int width, int top, const int32_t* pos, const float* wts, float* y, int E, const int32_t* ids, const void* x,
+                              int tokens, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     if (width <= 0 || top <= 0) return VK_BAD_SHAPE;
-    return launch_dependent(experts_combine_kernel, dim3(tokens), dim3(256), 0, stream, o, width, top, pos, wts, y);
+    if (dtype == 0)
+        return launch_dependent(experts_combine_kernel<float>, dim3(tokens), dim3(256), 0, stream, o, width, top, pos, wts, y, E, ids, (const float*)x);
+    return launch_dependent(experts_combine_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, o, width, top, pos, wts, y, E, ids,
+                            (const __nv_bfloat16*)x);
+}
+
+// x [tokens][width] in dtype; wr float32 [all][width], correction float32 [all] or null, all = experts + identities, in `count` equal groups of
+// neighbours of which `keep` take part; ids int32 [tokens][top], wts float32 [tokens][top].
+VK_API int vk_experts_route_scored(const void* x, int width, const float* wr, const float* correction, int all, int top, int count, int keep, float scale,
+                                   int32_t* ids, float* wts, int tokens, int dtype, cudaStream_t stream) {
+    if (tokens <= 0) return VK_OK;
+    if (width <= 0 || all <= 0 || count <= 0 || all % count || keep <= 0 || keep > count || top <= 0 || top > 32 || top > all / count * keep) return VK_BAD_SHAPE;
+    const int tb = tokens > 64 ? 4 : 1;
+    const size_t smem = (size_t)tb * (2 * all + count) * sizeof(float);
+    if (smem > 48 * 1024) return VK_TOO_LARGE;
+    const dim3 grid((tokens + tb - 1) / tb);
+#define VK_ERS(T, TB)                                                                                                                          \
+    return launch_dependent(experts_route_scored_kernel<T, TB>, grid, dim3(128), smem, stream, (const T*)x, width, wr, correction, all, top, count, \
+                            keep, scale, ids, wts, tokens)
+    if (dtype == 0) {
+        if (tb == 4) VK_ERS(float, 4);
+        VK_ERS(float, 1);
+    }
+    if (tb == 4) VK_ERS(__nv_bfloat16, 4);
+    VK_ERS(__nv_bfloat16, 1);
+#undef VK_ERS
 }
 
 // x [tokens][width] in dtype; wr float32 [E][width], br float32 [E] or null; ids int32 [tokens][top], wts float32 [tokens][top].
@@ -284,7 +407,7 @@ VK_API int vk_experts_route_table(const int32_t* tokens, const int32_t* table, i
 
 // wgu [E][2 ff][width] (an expert's gate rows, then its up rows) in dtype; out [tokens * top][ff] in dtype.  act: 0 none, 1 gelu (erf),
 // 2 gelu (tanh), 3 silu, 4 the clamped form min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).
-VK_API int vk_experts_gate_up(const void* x, int width, const void* wgu, int ff, int top, const int32_t* ids, int act, float limit, float alpha,
+VK_API int vk_experts_gate_up(const void* x, int width, const void* wgu, int ff, int top, const int32_t* ids, int E, int act, float limit, float alpha,
                               void* out, int tokens, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     if (width <= 0 || ff <= 0 || top <= 0 || act < 0 || act > 4 || (act == 4 && !(limit > 0.0f))) return VK_BAD_SHAPE;
@@ -294,24 +417,30 @@ VK_API int vk_experts_gate_up(const void* x, int width, const void* wgu, int ff,
     if (gy > 64) gy = 64;
     dim3 grid(tokens * top, gy);
     if (dtype == 0)
-        return launch_dependent(experts_gate_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, width, (const float*)wgu, ff, top, ids, act,
+        return launch_dependent(experts_gate_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, width, (const float*)wgu, ff, top, ids, E, act,
                                 limit, alpha, (float*)out);
     return launch_dependent(experts_gate_up_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, width,
-                            (const __nv_bfloat16*)wgu, ff, top, ids, act, limit, alpha, (__nv_bfloat16*)out);
+                            (const __nv_bfloat16*)wgu, ff, top, ids, E, act, limit, alpha, (__nv_bfloat16*)out);
 }
 
-// act [tokens * top][ff] and wd [E][width][ff] in dtype; y float32 [tokens][width] is added to.
-VK_API int vk_experts_down(const void* act, int ff, const void* wd, int width, int top, const int32_t* ids, const float* wts, float* y, int tokens,
-                           int dtype, cudaStream_t stream) {
+// act [tokens * top][ff] and wd [E][width][ff] in dtype; y float32 [tokens][width] is added to; ids of E and more: the token's row of x.
+VK_API int vk_experts_down(const void* act, int ff, const void* wd, int width, int top, const int32_t* ids, const float* wts, float* y, int E,
+                           const void* x, int tokens, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     if (width <= 0 || ff <= 0 || top <= 0) return VK_BAD_SHAPE;
     const size_t smem = (size_t)top * ff * sizeof(float);
-    if (smem > 48 * 1024) return VK_TOO_LARGE;
+    if (smem > 200 * 1024) return VK_TOO_LARGE;
     int gy = (width + 7) / 8;
     if (gy > 64) gy = 64;
     dim3 grid(tokens, gy);
+    if (smem > 48 * 1024) {
+        cudaError_t e = dtype == 0 ? cudaFuncSetAttribute(experts_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
+                                   : cudaFuncSetAttribute(experts_down_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
     if (dtype == 0)
-        return launch_dependent(experts_down_kernel<float>, grid, dim3(256), smem, stream, (const float*)act, ff, (const float*)wd, width, top, ids, wts, y);
+        return launch_dependent(experts_down_kernel<float>, grid, dim3(256), smem, stream, (const float*)act, ff, (const float*)wd, width, top, ids, wts, y,
+                                E, (const float*)x);
     return launch_dependent(experts_down_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)act, ff, (const __nv_bfloat16*)wd,
-                            width, top, ids, wts, y);
+                            width, top, ids, wts, y, E, (const __nv_bfloat16*)x);
 }

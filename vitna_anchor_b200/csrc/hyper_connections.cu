@@ -97,10 +97,11 @@ __global__ void embed_scaled_kernel(const T* __restrict__ table, const int32_t* 
     }
 }
 
-// 0: gelu, the erf form  0.5 z (1 + erf(z / sqrt 2));  1: gelu, the tanh form;  2: silu
+// 0: gelu, the erf form  0.5 z (1 + erf(z / sqrt 2));  1: gelu, the tanh form;  2: silu;  3: relu squared
 template <int KIND> __device__ __forceinline__ float activate(float z) {
     if (KIND == 0) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
     if (KIND == 1) return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
+    if (KIND == 3) { const float r = fmaxf(z, 0.0f); return r * r; }
     return z / (1.0f + expf(-z));
 }
 
@@ -171,6 +172,7 @@ static int launch_activation(const void* x, void* out, size_t n, int kind, cudaS
     if (kind == 0) activation_kernel<T, 0><<<grid, 256, 0, stream>>>((const T*)x, (T*)out, n);
     else if (kind == 1) activation_kernel<T, 1><<<grid, 256, 0, stream>>>((const T*)x, (T*)out, n);
     else if (kind == 2) activation_kernel<T, 2><<<grid, 256, 0, stream>>>((const T*)x, (T*)out, n);
+    else if (kind == 3) activation_kernel<T, 3><<<grid, 256, 0, stream>>>((const T*)x, (T*)out, n);
     else return VK_BAD_SHAPE;
     return launch_status();
 }

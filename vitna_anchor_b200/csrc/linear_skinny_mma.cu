@@ -46,7 +46,7 @@ struct MmaParams {
     const int32_t* slot;
     __nv_bfloat16* cache;
     int nh, nkv, hd, page_size;
-    int act;                     // ME_SAME: an activation on the float32 sums before they are rounded (activate_rt; 0 none); ME_SWIGLU: the gate's function (0: silu)
+    int act;                     // ME_SAME: an activation on the float32 sums before they are rounded (activate_dense; 0 none); ME_SWIGLU: the gate's function (0: silu)
 };
 
 __device__ __forceinline__ void mm_cp_async16(void* dst, const void* src) {
@@ -78,7 +78,7 @@ __device__ __forceinline__ void mma_finish(const MmaParams& p, int u, int r0, in
     typedef __nv_bfloat16 T;
     if (EPI == ME_SAME) {
         T* o = reinterpret_cast<T*>(p.out) + (size_t)m * p.N;
-        if (p.act) { a0 = activate_rt(p.act, a0); a1 = activate_rt(p.act, a1); }
+        if (p.act) { a0 = activate_dense(p.act, a0); a1 = activate_dense(p.act, a1); }
         o[r0] = __float2bfloat16_rn(a0);
         if (has1) o[r1] = __float2bfloat16_rn(a1);
     } else if (EPI == ME_F32) {
@@ -878,7 +878,7 @@ static int linear_skinny_mma_impl(const void* x, const int32_t* rows, const floa
                                   const float* sin_t, const int32_t* slot, void* cache, int nh, int nkv, int hd, int page_size, int act,
                                   cudaStream_t stream) {
     if (M <= 0 || N <= 0) return VK_OK;
-    if (K <= 0 || ldx < K || epi < 0 || epi > 4 || K % 32 != 0 || act < 0 || act > 3 || (act && epi != ME_SAME && epi != ME_SWIGLU)) return VK_BAD_SHAPE;
+    if (K <= 0 || ldx < K || epi < 0 || epi > 4 || K % 32 != 0 || act < 0 || act > 4 || (act && epi != ME_SAME && epi != ME_SWIGLU)) return VK_BAD_SHAPE;
     if (M > 64) return VK_TOO_LARGE;
     if (((uintptr_t)w % 16) || ((uintptr_t)x % 16)) return VK_BAD_ALIGNMENT;
     if (norm_w ? (ldx % 4 != 0 || ((uintptr_t)norm_w % 16)) : (ldx % 8 != 0)) return VK_BAD_ALIGNMENT;
@@ -901,7 +901,7 @@ VK_API int vk_linear_skinny_mma(const void* x, const int32_t* rows, const float*
                                   page_size, 0, stream);
 }
 
-// out (bfloat16) = act(x' @ w.T) for at most 64 rows: the activation (activate_rt) on the float32 sums in the epilogue.
+// out (bfloat16) = act(x' @ w.T) for at most 64 rows: the activation (activate_dense) on the float32 sums in the epilogue.
 VK_API int vk_linear_skinny_mma_act(const void* x, const int32_t* rows, const float* norm_w, float eps, const void* w, void* out,
                                     int M, int N, int K, int ldx, int act, cudaStream_t stream) {
     return linear_skinny_mma_impl(x, rows, norm_w, eps, w, out, M, N, K, ldx, ME_SAME, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 0, 0, 0,
@@ -912,7 +912,7 @@ VK_API int vk_linear_skinny_mma_act(const void* x, const int32_t* rows, const fl
 // numbers them (the gate's function on the rounded sums, in the epilogue).
 VK_API int vk_linear_skinny_mma_gated(const void* x, const int32_t* rows, const float* norm_w, float eps, const void* w, void* out,
                                       int M, int N, int K, int ldx, int act, cudaStream_t stream) {
-    if (act < 1) return VK_BAD_SHAPE;
+    if (act < 1 || act > 3) return VK_BAD_SHAPE;
     return linear_skinny_mma_impl(x, rows, norm_w, eps, w, out, M, N, K, ldx, ME_SWIGLU, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 0, 0, 0,
                                   act, stream);
 }

@@ -47,7 +47,7 @@ struct TcExtra {
     const int32_t* slot;
     __nv_bfloat16* cache;
     int nh, nkv, hd, page_size;
-    int act;                     // TC_SAME: an activation on the float32 sums before they are rounded (activate_rt; 0 none)
+    int act;                     // TC_SAME: an activation on the float32 sums before they are rounded (activate_dense; 0 none)
     // Products of groups of rows with a weight matrix each (a routed feed-forward's experts): the weight is group_rows rows a group,
     // one group after another, and row tile number i of x belongs to group tile_group[i] (negative: the tile has no rows and its
     // blocks leave at once).  The table is the output of a kernel before this one.  Null: one weight matrix for all rows.
@@ -313,7 +313,7 @@ __global__ void __launch_bounds__(TC_THREADS) linear_tcgen05_kernel(const __grid
                     __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * N + col;
                     if (ex.act) {
 #pragma unroll
-                        for (int j = 0; j < 32; j++) r[j] = __float_as_uint(activate_rt(ex.act, __uint_as_float(r[j])));
+                        for (int j = 0; j < 32; j++) r[j] = __float_as_uint(activate_dense(ex.act, __uint_as_float(r[j])));
                     }
                     if (whole && (N % 8 == 0)) {
 #pragma unroll
@@ -618,7 +618,7 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
                             __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * N + col;
                             if (ex.act) {
 #pragma unroll
-                                for (int q = 0; q < 32; q++) r[q] = __float_as_uint(activate_rt(ex.act, __uint_as_float(r[q])));
+                                for (int q = 0; q < 32; q++) r[q] = __float_as_uint(activate_dense(ex.act, __uint_as_float(r[q])));
                             }
                             if (whole && (N % 8 == 0)) {
 #pragma unroll
@@ -771,7 +771,7 @@ using namespace vk;
 static int linear_tcgen05_impl(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int mode, int act, int* error,
                                cudaStream_t stream) {
     if (M <= 0 || N <= 0) return VK_OK;
-    if (K <= 0 || ldx < K || mode < 0 || mode > 2 || !error || act < 0 || act > 3 || (act && mode != 0)) return VK_BAD_SHAPE;
+    if (K <= 0 || ldx < K || mode < 0 || mode > 2 || !error || act < 0 || act > 4 || (act && mode != 0)) return VK_BAD_SHAPE;
     TcExtra ex{};
     ex.act = act;
     if (K % 8 != 0 || ldx % 8 != 0) return VK_BAD_SHAPE;
@@ -804,7 +804,7 @@ VK_API int vk_linear_tcgen05(const void* x, const void* w, void* out, int M, int
     return linear_tcgen05_impl(x, w, out, M, N, K, ldx, mode, 0, error, stream);
 }
 
-// out (bfloat16) = act(x @ w.T): the activation (activate_rt: 1 gelu erf, 2 gelu tanh, 3 silu) on the float32 sums in the epilogue.
+// out (bfloat16) = act(x @ w.T): the activation (activate_dense: 1 gelu erf, 2 gelu tanh, 3 silu, 4 relu squared) on the float32 sums in the epilogue.
 VK_API int vk_linear_tcgen05_act(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int act, int* error,
                                  cudaStream_t stream) {
     return linear_tcgen05_impl(x, w, out, M, N, K, ldx, 0, act, error, stream);

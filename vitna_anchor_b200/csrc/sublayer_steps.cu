@@ -7,6 +7,8 @@
 //                     Without w nothing is added: y is zeroed and xc written, which is how a pass begins.
 //                     One block a row; what a sublayer ADDED into the zeroed y is normed, scaled and summed into the float32
 //                     residual row, y is zero again for the next sublayer, and the next sublayer's input is written.
+//  pass_input         cat[t] = [ x[t] | x0[t] ] in the compute dtype, the input of the product that begins a pass over looped layers: the left
+//                     half from x, or the right half, or both (x is x0 then).
 //  glu_clamped        out = g' sigmoid(alpha g') (u' + 1),  g' = min(g, L),  u' = clamp(u, -L, L);  gu [T, 2I] -> out [T, I].
 //
 // All arithmetic is float32; accurate expf, division and sqrtf.
@@ -263,9 +265,40 @@ __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ 
     }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(256) pass_input_kernel(const float* __restrict__ x, T* __restrict__ cat, int n, int left, int right, int vec) {
+    dependency_wait();
+    let_dependents_start();
+    const float* in = x + (size_t)blockIdx.x * n;
+    T* out = cat + (size_t)blockIdx.x * 2 * n;
+    if (vec) {
+        for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(in + i);
+            if (left) sw_store4<T>(out + i, v.x, v.y, v.z, v.w);
+            if (right) sw_store4<T>(out + n + i, v.x, v.y, v.z, v.w);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const T v = from_f32<T>(in[i]);
+        if (left) out[i] = v;
+        if (right) out[n + i] = v;
+    }
+}
+
 }  // namespace vk
 
 using namespace vk;
+
+// x float32 [rows][n]; cat [rows][2 n] in dtype: its left and / or right half is written.
+VK_API int vk_pass_input(const float* x, void* cat, int rows, int n, int left, int right, int dtype, cudaStream_t stream) {
+    if (rows <= 0) return VK_OK;
+    if (n <= 0) return VK_BAD_SHAPE;
+    const int vec = n % 4 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)cat % 16) == 0;
+    if (dtype == 0) return launch_dependent(pass_input_kernel<float>, dim3(rows), dim3(256), 0, stream, x, (float*)cat, n, left, right, vec);
+    return launch_dependent(pass_input_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, x, (__nv_bfloat16*)cat, n, left, right, vec);
+}
+
 
 // table [vocab][hidden], second [buckets + 1][hidden] (null: no second row) in dtype; last_token int32 [slots] (may be null when
 // second is null); x float32 [tokens][hidden]; xc [tokens][hidden] in dtype or null.

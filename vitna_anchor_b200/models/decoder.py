@@ -12,6 +12,9 @@ convolution in front of an attention): it says so with state_spec(), and its
 run names a second cache layer (`state`) that holds it; the mixer then sees
 one view with both.  A token input with state_spec() (the token before a
 step's first one) gets a cache layer of its own behind all others.
+
+A run may name a part that changes the residual stream right before its block (`before`: what a pass over looped layers begins
+with).  Such a part sees the embedding output once, right after it is made (remember), and is then called before its runs.
 """
 from __future__ import annotations
 
@@ -30,6 +33,7 @@ class LayerRun:
     cache: int                  # cache layer this run uses
     write_cache: bool = True    # False: read what another run of the step wrote
     state: int = -1             # cache layer of the fixed-size state the mixer keeps beside its pages (-1: none)
+    before: Optional[Part] = None       # changes the residual rows ahead of the block: before.forward(x, ctx, at_embedding)
 
 
 class DecoderModel:
@@ -63,6 +67,10 @@ class DecoderModel:
         for c, n in enumerate(writers):
             if specs[c] is not None and n != 1:
                 raise ValueError(f"cache layer {c} has {n} writers in the schedule; it needs exactly one")
+        self.entries: List[Part] = []                       # the parts that runs begin with, each once
+        for run in self.schedule:
+            if run.before is not None and all(run.before is not e for e in self.entries):
+                self.entries.append(run.before)
         self._input_state = -1
         beside = embedding.state_spec() if hasattr(embedding, "state_spec") else None
         if beside is not None:
@@ -74,13 +82,14 @@ class DecoderModel:
         return list(self._cache_specs)
 
     def parts(self) -> List[Part]:
-        return [self.embedding, *self.blocks, self.final_norm, self.lm_head] + ([self.collect] if self.collect is not None else [])
+        return [self.embedding, *self.blocks, self.final_norm, self.lm_head] + ([self.collect] if self.collect is not None else []) + self.entries
 
     def step_weight_bytes(self) -> int:
         """Bytes of weights a decode step reads: every block as often as it runs, the output matrix once,
         and one embedding row per token (not counted)."""
         per_block = [b.weight_bytes() for b in self.blocks]
-        return sum(per_block[r.block] for r in self.schedule) + self.final_norm.weight_bytes() + self.lm_head.weight_bytes()
+        entries = sum(r.before.weight_bytes() for r in self.schedule if r.before is not None)
+        return entries + sum(per_block[r.block] for r in self.schedule) + self.final_norm.weight_bytes() + self.lm_head.weight_bytes()
 
     @property
     def capture_safe(self) -> bool:
@@ -98,7 +107,11 @@ class DecoderModel:
         x = self.embedding.forward(ctx) if self._input_state < 0 else self.embedding.forward(ctx, ctx.caches[self._input_state].state)
         if self.position is not None:
             self.position.on_embeddings(x, ctx)
+        for part in self.entries:
+            part.remember(x, ctx)
         for i, run in enumerate(self.schedule):
+            if run.before is not None:
+                run.before.forward(x, ctx, i == 0)
             cache = ctx.caches[run.cache] if run.cache >= 0 else None
             if run.state >= 0:
                 cache = replace(cache, state=ctx.caches[run.state].state)

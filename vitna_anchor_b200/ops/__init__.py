@@ -692,17 +692,18 @@ def attention(q: torch.Tensor, pages: torch.Tensor, meta, ctx, out: torch.Tensor
 # ---------------------------------------------------------------------------
 
 ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2}
+DENSE_ACTIVATIONS = {**ACTIVATIONS, "relu2": 3}         # where no second product is gated: relu squared too
 
 
 def activation(x: torch.Tensor, kind: str, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out = act(x) element by element (in place unless out is given); kind: gelu (the erf form), gelu_tanh, silu."""
-    if kind not in ACTIVATIONS:
-        raise KernelError(f"activation: {kind!r} is not one of {sorted(ACTIVATIONS)}")
+    """out = act(x) element by element (in place unless out is given); kind: gelu (the erf form), gelu_tanh, silu, relu2."""
+    if kind not in DENSE_ACTIVATIONS:
+        raise KernelError(f"activation: {kind!r} is not one of {sorted(DENSE_ACTIVATIONS)}")
     out = x if out is None else out
     _req(x, "x"); _req(out, "out", x.dtype)
     if out.numel() != x.numel():
         raise KernelError("activation: sizes differ")
-    _check(lib().vk_activation(_p(x), _p(out), ctypes.c_size_t(x.numel()), ACTIVATIONS[kind], _dt(x), _stream()), "activation")
+    _check(lib().vk_activation(_p(x), _p(out), ctypes.c_size_t(x.numel()), DENSE_ACTIVATIONS[kind], _dt(x), _stream()), "activation")
     return out
 
 
@@ -786,6 +787,13 @@ def qk_norm_store(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opti
     return q_out
 
 
+def _out_rows(out: torch.Tensor, dtype: torch.dtype, rows: int, width: int, name: str) -> int:
+    """The distance in elements between the rows of an attention's output, which may be columns of a wider matrix."""
+    if not out.is_cuda or out.dtype != dtype or out.dim() != 2 or out.shape != (rows, width) or out.stride(1) != 1:
+        raise KernelError(f"{name}: out is not a CUDA matrix [tokens, heads * v_dim] of the queries' dtype with unit column stride")
+    return max(out.stride(0), width)
+
+
 def attention_rows_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_tables: torch.Tensor, token_seg: torch.Tensor,
                           positions: torch.Tensor, out: torch.Tensor, nh: int, nkv: int, hd: int, vd: int, page_size: int, scale: float,
                           window: int = 0, dist_bias: Optional[torch.Tensor] = None, tok_list: Optional[torch.Tensor] = None,
@@ -795,9 +803,10 @@ def attention_rows_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_tabl
     v_in_key: the cache holds keys alone and a key's first vd values are its value.  v_share > 1: that many neighbouring
     key heads read one value head (two score maps over the same values)."""
     _req(q, "q", dims=2); _req(cache_layer, "cache_layer", q.dtype); _req(block_tables, "block_tables", torch.int32, 2)
-    _req(token_seg, "token_seg", torch.int32, 1); _req(positions, "positions", torch.int32, 1); _req(out, "out", q.dtype, 2)
+    _req(token_seg, "token_seg", torch.int32, 1); _req(positions, "positions", torch.int32, 1)
     T = q.shape[0]
-    if q.shape[1] != nh * hd or out.shape != (T, nh * vd) or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size:
+    out_ld = _out_rows(out, q.dtype, T, nh * vd, "attention_rows_biased")
+    if q.shape[1] != nh * hd or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size:
         raise KernelError("attention_rows_biased: shapes do not fit the head counts")
     if token_seg.shape[0] != T or positions.shape[0] != T:
         raise KernelError("attention_rows_biased: per-token arrays differ in length")
@@ -811,7 +820,7 @@ def attention_rows_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_tabl
         n = tok_list.shape[0]
     _check(lib().vk_attention_rows_biased(_p(q), _p(cache_layer), _p(block_tables), _p(token_seg), _p(positions), _p(tok_list), _p(out), n, nh,
                                           nkv, hd, vd, page_size, block_tables.shape[1], ctypes.c_float(scale), window, _p(dist_bias),
-                                          0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), _dt(q), _stream()),
+                                          0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _dt(q), _stream()),
            "attention_rows_biased")
     return out
 
@@ -899,10 +908,11 @@ def attention_decode_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_ta
     """The split-key attention of single decoded tokens in the unrotated form: values of size vd, an optional bias by distance.
     scratch: attention_decode_scratch_bytes(scratch_tokens, nh, nkv, max(hd, vd), max_context) bytes, zero at first use."""
     _req(q, "q", dims=2); _req(cache_layer, "cache_layer", q.dtype); _req(block_tables, "block_tables", torch.int32, 2)
-    _req(token_seg, "token_seg", torch.int32, 1); _req(positions, "positions", torch.int32, 1); _req(out, "out", q.dtype, 2)
+    _req(token_seg, "token_seg", torch.int32, 1); _req(positions, "positions", torch.int32, 1)
     _req(scratch, "scratch", torch.uint8, 1)
     T = q.shape[0]
-    if q.shape[1] != nh * hd or out.shape != (T, nh * vd) or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size:
+    out_ld = _out_rows(out, q.dtype, T, nh * vd, "attention_decode_biased")
+    if q.shape[1] != nh * hd or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size:
         raise KernelError("attention_decode_biased: shapes do not fit the head counts")
     if dist_bias is not None:
         _req(dist_bias, "dist_bias", torch.float32, 2)
@@ -917,7 +927,7 @@ def attention_decode_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_ta
     _check(lib().vk_attention_decode_biased(_p(q), _p(cache_layer), _p(block_tables), _p(token_seg), _p(positions), _p(tok_list), _p(out),
                                             _p(scratch), scratch_tokens, n, nh, nkv, hd, vd, page_size, block_tables.shape[1], max_context,
                                             grid_context, ctypes.c_float(scale), window, _p(dist_bias),
-                                            0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), _dt(q), _stream()),
+                                            0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _dt(q), _stream()),
            "attention_decode_biased")
     return out
 
@@ -931,8 +941,9 @@ def attention_prefill_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_t
     """Causal attention of prompt portions in bfloat16 on the tensor cores, in the unrotated form.  tiles int32 [n, 4]: first
     token, rows (1..64), position of the first token, segment."""
     _req(q, "q", torch.bfloat16, 2); _req(cache_layer, "cache_layer", torch.bfloat16)
-    _req(block_tables, "block_tables", torch.int32, 2); _req(tiles, "tiles", torch.int32, 2); _req(out, "out", torch.bfloat16, 2)
-    if (q.shape[1] != nh * hd or out.shape != (q.shape[0], nh * vd) or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size
+    _req(block_tables, "block_tables", torch.int32, 2); _req(tiles, "tiles", torch.int32, 2)
+    out_ld = _out_rows(out, torch.bfloat16, q.shape[0], nh * vd, "attention_prefill_biased")
+    if (q.shape[1] != nh * hd or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size
             or tiles.shape[1] != 4):
         raise KernelError("attention_prefill_biased: shapes do not fit the head counts")
     if hd not in BIASED_PREFILL_HEAD_SIZES or vd not in BIASED_PREFILL_HEAD_SIZES:
@@ -943,7 +954,7 @@ def attention_prefill_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_t
             raise KernelError("attention_prefill_biased: the bias table is not [distances, heads]")
     _check(lib().vk_attention_prefill_biased(_p(q), _p(cache_layer), _p(block_tables), _p(tiles), _p(out), tiles.shape[0], nh, nkv, hd, vd,
                                              page_size, block_tables.shape[1], ctypes.c_float(scale), window, _p(dist_bias),
-                                             0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), _stream()), "attention_prefill_biased")
+                                             0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _stream()), "attention_prefill_biased")
     return out
 
 
@@ -959,7 +970,8 @@ def attention_biased(q: torch.Tensor, pages: torch.Tensor, meta, ctx, out: torch
     dec_ok = (bool(ctx.num_dec) and not exact and hd % vec == 0 and vd % vec == 0 and max(hd, vd) <= 256 and vd // vec <= 32
               and ctx.workspace.max_context <= 128 * 256)
     pre_ok = (bool(ctx.num_pre) and q.dtype == torch.bfloat16 and hd in BIASED_PREFILL_HEAD_SIZES and vd in BIASED_PREFILL_HEAD_SIZES
-              and ctx.pre_tiles is not None and q.data_ptr() % 16 == 0 and pages.data_ptr() % 16 == 0)
+              and ctx.pre_tiles is not None and q.data_ptr() % 16 == 0 and pages.data_ptr() % 16 == 0 and out.data_ptr() % 4 == 0
+              and out.stride(0) % 2 == 0)
     rows = lambda toks: attention_rows_biased(q, pages, meta.block_tables, ctx.token_seg, ctx.positions, out, nh, nkv, hd, vd, page_size,
                                               scale, window, dist_bias, toks, v_in_key, v_share)
     if dec_ok:
@@ -981,15 +993,15 @@ def attention_biased(q: torch.Tensor, pages: torch.Tensor, meta, ctx, out: torch
 
 
 def linear_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tensor:
-    """out = act(x @ w.T) in x's dtype; kind one of ACTIVATIONS.  In bfloat16 the activation is the epilogue of the few-rows
+    """out = act(x @ w.T) in x's dtype; kind one of DENSE_ACTIVATIONS.  In bfloat16 the activation is the epilogue of the few-rows
     tensor-core product (up to 64 rows) or of the tcgen05 product, on the float32 sums; elsewhere it is a launch of its own."""
-    if kind not in ACTIVATIONS:
-        raise KernelError(f"linear_act: {kind!r} is not one of {sorted(ACTIVATIONS)}")
+    if kind not in DENSE_ACTIVATIONS:
+        raise KernelError(f"linear_act: {kind!r} is not one of {sorted(DENSE_ACTIVATIONS)}")
     M, K = x.shape
     N = w.shape[0]
     if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K and tuple(out.shape) == (M, N) and out.dtype == x.dtype:
         _req(w, "w", torch.bfloat16, 2); _req(out, "out", torch.bfloat16, 2)
-        act = ACTIVATIONS[kind] + 1
+        act = DENSE_ACTIVATIONS[kind] + 1
         if (skinny_takes(x.dtype, M, K, N) and K % 32 == 0 and x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
                 and w.data_ptr() % 16 == 0):
             ldx = x.stride(0) if M > 1 else max(K, x.stride(0))
@@ -1376,6 +1388,22 @@ def experts_route(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional[to
     _check(lib().vk_experts_route(_p(x), W, _p(w_router), _p(b_router), w_router.shape[0], top, _p(ids), _p(wts), T, _dt(x), _stream()), "experts_route")
 
 
+def experts_route_scored(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int, scale: float,
+                         ids: torch.Tensor, wts: torch.Tensor) -> None:
+    """s = softmax(w_router x) over all rows of w_router (experts, then identities); of `groups` equal groups of neighbours the `keep` with the largest
+    s + correction; of their members the `top` with the largest s + correction go to ids [T, top], s / (sum of the chosen + 1e-20) * scale to
+    wts [T, top]."""
+    _req(x, "x", dims=2); _req(w_router, "w_router", torch.float32, 2); _req(ids, "ids", torch.int32, 2); _req(wts, "wts", torch.float32, 2)
+    T, W = x.shape
+    E = w_router.shape[0]
+    if w_router.shape[1] != W or ids.shape != (T, top) or wts.shape != (T, top) or (correction is not None and correction.shape != (E,)):
+        raise KernelError("experts_route_scored: shapes do not fit")
+    if correction is not None:
+        _req(correction, "correction", torch.float32, 1)
+    _check(lib().vk_experts_route_scored(_p(x), W, _p(w_router), _p(correction), E, top, groups, keep, ctypes.c_float(scale), _p(ids), _p(wts), T, _dt(x),
+                                         _stream()), "experts_route_scored")
+
+
 def experts_route_table(tokens: torch.Tensor, table: torch.Tensor, E: int, top: int, ids: torch.Tensor, wts: torch.Tensor) -> None:
     """ids [T, top] = table[token id, :top] (int32 [vocab, >= top]); every weight 1 / top."""
     _req(tokens, "tokens", torch.int32, 1); _req(table, "table", torch.int32, 2); _req(ids, "ids", torch.int32, 2); _req(wts, "wts", torch.float32, 2)
@@ -1396,7 +1424,7 @@ def _expert_act(activation: str, what: str) -> int:
 
 def experts_apply(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, act_buf: torch.Tensor,
                   y: torch.Tensor, activation: str = "silu", limit: float = 0.0, alpha: float = 1.702) -> torch.Tensor:
-    """y [T, W] (float32) += sum_k wts[t, k] W_down,e (act(W_gate,e x) * W_up,e x), e = ids[t, k]; w_gate_up [E, 2 ff, W], w_down [E, W, ff]
+    """y [T, W] (float32) += sum_k wts[t, k] W_down,e (act(W_gate,e x) * W_up,e x), e = ids[t, k] (an id of E or more: x itself); w_gate_up [E, 2 ff, W], w_down [E, W, ff]
     in x's dtype; act_buf [T * top, ff] in x's dtype.  activation "clamped": min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u) + 1)."""
     _req(x, "x", dims=2); _req(w_gate_up, "w_gate_up", x.dtype, 3); _req(w_down, "w_down", x.dtype, 3); _req(y, "y", torch.float32, 2)
     _req(act_buf, "act_buf", x.dtype, 2)
@@ -1406,9 +1434,9 @@ def experts_apply(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor
     if w_gate_up.shape != (E, 2 * ff, W) or w_down.shape != (E, W, ff) or y.shape != (T, W) or act_buf.shape != (T * top, ff):
         raise KernelError("experts_apply: shapes do not fit")
     act = _expert_act(activation, "experts_apply")
-    _check(lib().vk_experts_gate_up(_p(x), W, _p(w_gate_up), ff, top, _p(ids), act, ctypes.c_float(limit), ctypes.c_float(alpha), _p(act_buf), T,
+    _check(lib().vk_experts_gate_up(_p(x), W, _p(w_gate_up), ff, top, _p(ids), E, act, ctypes.c_float(limit), ctypes.c_float(alpha), _p(act_buf), T,
                                     _dt(x), _stream()), "experts_gate_up")
-    _check(lib().vk_experts_down(_p(act_buf), ff, _p(w_down), W, top, _p(ids), _p(wts), _p(y), T, _dt(x), _stream()), "experts_down")
+    _check(lib().vk_experts_down(_p(act_buf), ff, _p(w_down), W, top, _p(ids), _p(wts), _p(y), E, _p(x), T, _dt(x), _stream()), "experts_down")
     return y
 
 
@@ -1463,7 +1491,7 @@ def experts_apply_grouped(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torc
                                                _stream()), "linear_tcgen05_grouped")
     _check(lib().vk_linear_tcgen05_grouped(_p(act_buf), _p(w_down), _p(o), rows, W, ff, ff, E, _p(tile_group), 1, 0, 0, _p(error_word()),
                                            _stream()), "linear_tcgen05_grouped")
-    _check(lib().vk_experts_combine(_p(o), W, top, _p(pos), _p(wts), _p(y), T, _stream()), "experts_combine")
+    _check(lib().vk_experts_combine(_p(o), W, top, _p(pos), _p(wts), _p(y), E, _p(ids), _p(x), T, _dt(x), _stream()), "experts_combine")
     return y
 
 
@@ -1556,13 +1584,15 @@ def gla(proj: torch.Tensor, a_off: int, a2t: torch.Tensor, bias: torch.Tensor, t
 
 def mixed_attn_prepare(proj: torch.Tensor, positions: torch.Tensor, slot_mapping: Optional[torch.Tensor], q_norm: Optional[torch.Tensor],
                        k_norm: Optional[torch.Tensor], eps: float, freq: Optional[torch.Tensor], dims: int, vfreq: Optional[torch.Tensor],
-                       q_out: torch.Tensor, cache_layer: Optional[torch.Tensor], nh: int, nkv: int, hd: int, vd: int, page_size: int) -> torch.Tensor:
-    """From the float32 row [q | k | v] of the first product: q and k heads / rms * weight (eps < 0: no norm), the first `dims` values turned
+                       q_out: torch.Tensor, cache_layer: Optional[torch.Tensor], nh: int, nkv: int, hd: int, vd: int, page_size: int,
+                       bias: Optional[torch.Tensor] = None, v_mult: float = 1.0, off: int = 0) -> torch.Tensor:
+    """From the columns [q | k | v] at `off` of the first product's float32 rows, plus `bias` [its columns] if given: q and k heads / rms * weight (eps < 0: no norm),
+    v times v_mult, the first `dims` values of q and k turned
     in pairs (i, i + dims / 2) by position * freq[i]; v turned over all its pairs by position * vfreq[m] (None: not); q to q_out, k and v
     into the layer's pages at slot_mapping (-1: no write)."""
     _req(proj, "proj", torch.float32, 2); _req(positions, "positions", torch.int32, 1); _req(q_out, "q_out", dims=2)
     T, N = proj.shape
-    if N < (nh + nkv) * hd + nkv * vd or q_out.shape != (T, nh * hd) or positions.shape[0] < T:
+    if off < 0 or N < off + (nh + nkv) * hd + nkv * vd or q_out.shape != (T, nh * hd) or positions.shape[0] < T:
         raise KernelError("mixed_attn_prepare: shapes do not fit the head counts")
     for v, n, name in ((q_norm, hd, "q_norm"), (k_norm, hd, "k_norm"), (freq, dims // 2, "freq"), (vfreq, vd // 2, "vfreq")):
         if v is not None:
@@ -1571,13 +1601,17 @@ def mixed_attn_prepare(proj: torch.Tensor, positions: torch.Tensor, slot_mapping
                 raise KernelError(f"mixed_attn_prepare: {name} has {v.shape[0]} values, expected {n}")
     if dims and freq is None:
         raise KernelError("mixed_attn_prepare: a rotation needs its frequencies")
+    if bias is not None:
+        _req(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != (nh + nkv) * hd + nkv * vd:
+            raise KernelError("mixed_attn_prepare: the bias does not fit the head counts")
     if cache_layer is not None:
         _req(cache_layer, "cache_layer", q_out.dtype); _req(slot_mapping, "slot_mapping", torch.int32, 1)
         if _page_size_of(cache_layer, nkv, hd, vd) != page_size or slot_mapping.shape[0] < T:
             raise KernelError("mixed_attn_prepare: the cache layer does not fit the page size")
-    _check(lib().vk_mixed_attn_prepare(_p(proj), N, _p(positions), _p(slot_mapping if cache_layer is not None else None), _p(q_norm), _p(k_norm),
+    _check(lib().vk_mixed_attn_prepare(ctypes.c_void_p(proj.data_ptr() + 4 * off), N, _p(positions), _p(slot_mapping if cache_layer is not None else None), _p(q_norm), _p(k_norm),
                                        ctypes.c_float(eps), _p(freq if dims else None), dims, _p(vfreq), _p(q_out), _p(cache_layer), T, nh, nkv, hd, vd,
-                                       page_size, _dt(q_out), _stream()), "mixed_attn_prepare")
+                                       page_size, _p(bias), ctypes.c_float(v_mult), _dt(q_out), _stream()), "mixed_attn_prepare")
     return q_out
 
 
@@ -1711,4 +1745,82 @@ def latent_expand_gate(lat: torch.Tensor, w: torch.Tensor, gates: Optional[torch
         if gates.shape[0] != T:
             raise KernelError("latent_expand_gate: the gates do not fit the tokens")
     _check(lib().vk_latent_expand_gate(_p(lat), _p(w), _p(gates), N, gate_off, H, rank, vd, _p(out), T, _dt(lat), _stream()), "latent_expand_gate")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# A product in front of a pass over looped layers; the state-space mixer
+# ---------------------------------------------------------------------------
+
+def pass_input(x: torch.Tensor, cat: torch.Tensor, left: bool, right: bool) -> torch.Tensor:
+    """cat [T, 2 W]: its left and / or right half <- x (float32 [T, W]) in cat's dtype."""
+    _req(x, "x", torch.float32, 2); _req(cat, "cat", dims=2)
+    T, W = x.shape
+    if cat.shape != (T, 2 * W):
+        raise KernelError("pass_input: cat is not [tokens, 2 * width]")
+    _check(lib().vk_pass_input(_p(x), _p(cat), T, W, int(left), int(right), _dt(cat), _stream()), "pass_input")
+    return cat
+
+
+def ssd_state_floats(H: int, G: int, N: int, P: int, taps: int) -> int:
+    """A slot's state: S [H, N, P], then the last taps - 1 inputs of the convolution, rounded up to a multiple of four."""
+    return (H * N * P + (taps - 1) * (H * P + 2 * G * N) + 3) // 4 * 4
+
+
+def ssd_max_state() -> int:
+    return int(lib().vk_ssd_max_state())
+
+
+def ssd_max_taps() -> int:
+    return int(lib().vk_ssd_max_taps())
+
+
+def ssd_chunked_scratch_bytes(tokens: int, segments: int, H: int, N: int, P: int) -> int:
+    fn = lib().vk_ssd_chunked_scratch_bytes
+    fn.restype = ctypes.c_size_t
+    return int(fn(tokens, segments, H, N, P))
+
+
+def ssd(proj: torch.Tensor, off: int, conv_w: torch.Tensor, conv_b: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor, D: torch.Tensor,
+        norm_w: torch.Tensor, eps: float, parts: int, mult: float, ctx, state: torch.Tensor, xbc: torch.Tensor, gates: torch.Tensor, y: torch.Tensor,
+        out: torch.Tensor, H: int, G: int, N: int, P: int, taps: int, chunk_scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The state-space mixer on a batch of segments, from the projections to the input of the output product.  proj float32 [T, *] with
+    z [H P] | x [H P] | B [G N] | C [G N] | dt [H] at columns off ..; state float32 [slots, ssd_state_floats], read and moved on; xbc [T, H P + 2 G N] (out's
+    dtype), gates [T, 2 H] and y [T, H P] (float32) are scratch; out [T, H P] (columns of a wider matrix allowed) = mult * (y silu(z)) / rms in
+    `parts` equal parts * norm_w.  Steps of single tokens take one launch for convolution, gates and step (not in the exact 32-bit routing);
+    bfloat16 with chunk_scratch (uint8, ssd_chunked_scratch_bytes) the chunked form; else token after token."""
+    inner, C = H * P, H * P + 2 * G * N
+    for name, t, d in (("proj", proj, 2), ("conv_w", conv_w, 2), ("dt_bias", dt_bias, 1), ("a_log", a_log, 1), ("D", D, 1), ("norm_w", norm_w, 1),
+                       ("state", state, 2), ("gates", gates, 2), ("y", y, 2)):
+        _req(t, name, torch.float32, d)
+    _req(xbc, "xbc", out.dtype, 2)
+    if conv_b is not None:
+        _req(conv_b, "conv_b", torch.float32, 1)
+    T, width = proj.shape
+    out_ld = _out_rows(out, out.dtype, T, inner, "ssd")
+    if (off < 0 or off + inner + C + H > width or conv_w.shape != (C, taps) or (conv_b is not None and conv_b.shape[0] != C) or dt_bias.shape[0] != H
+            or a_log.shape[0] != H or D.shape[0] != H or norm_w.shape[0] != inner or state.shape[1] != ssd_state_floats(H, G, N, P, taps)
+            or xbc.shape != (T, C) or gates.shape != (T, 2 * H) or y.shape != (T, inner)):
+        raise KernelError("ssd: shapes do not fit the head counts")
+    L, z_off, x_off, dt_off = lib(), off, off + inner, off + inner + C
+    stride = ctypes.c_size_t(state.stride(0))
+    exact = out.dtype == torch.float32 and _float32_exact
+    if ctx.decode_only and not exact:
+        _check(L.vk_ssd_decode(_p(proj), width, x_off, dt_off, _p(conv_w), _p(conv_b), _p(dt_bias), _p(a_log), _p(D), _p(ctx.seg_starts), _p(ctx.seg_slots),
+                               _p(state), stride, _p(y), ctx.num_segments, H, G, N, P, taps, _dt(out), _stream()), "ssd_decode")
+    else:
+        _check(L.vk_ssd_prepare(_p(proj), width, x_off, dt_off, _p(conv_w), _p(conv_b), _p(dt_bias), _p(a_log), _p(ctx.token_seg), _p(ctx.seg_starts),
+                                _p(ctx.seg_slots), _p(state), stride, _p(xbc), _p(gates), T, H, G, N, P, taps, _dt(out), _stream()), "ssd_prepare")
+        if chunk_scratch is not None and out.dtype == torch.bfloat16:
+            _req(chunk_scratch, "chunk_scratch", torch.uint8, 1)
+            if chunk_scratch.numel() < ssd_chunked_scratch_bytes(T, ctx.num_segments, H, N, P):
+                raise KernelError("ssd: the scratch of the chunked form is too small")
+            _check(L.vk_ssd_chunked(_p(xbc), _p(gates), _p(D), _p(ctx.seg_starts), _p(ctx.seg_slots), _p(state), stride, _p(y), _p(chunk_scratch),
+                                    ctx.num_segments, T, H, G, N, P, _stream()), "ssd_chunked")
+            add_launches(2)                             # three kernels
+        else:
+            _check(L.vk_ssd_recurrence(_p(xbc), _p(gates), _p(D), _p(ctx.seg_starts), _p(ctx.seg_slots), _p(state), stride, _p(y), ctx.num_segments, H, G,
+                                       N, P, _dt(out), _stream()), "ssd_recurrence")
+    _check(L.vk_ssd_gate(_p(y), _p(proj), width, z_off, x_off, _p(norm_w), ctypes.c_float(eps), ctypes.c_float(mult), parts, _p(out), out_ld,
+                         _p(ctx.token_seg), _p(ctx.seg_starts), _p(ctx.seg_slots), _p(state), stride, T, H, G, N, P, taps, _dt(out), _stream()), "ssd_gate")
     return out

@@ -4,7 +4,7 @@ The gate and up matrices are stacked by rows so that one product reads xn once.
 
 With another activation than silu (`activation`, one of ops.ACTIVATIONS) it is the same gated form, y = W_down (act(W_gate xn) * (W_up xn)).
 
-The dense feed-forward: y = W_down act(W_up xn), act one of ops.ACTIVATIONS (the erf or the tanh form of gelu, silu), or "xielu":
+The dense feed-forward: y = W_down act(W_up xn), act one of ops.DENSE_ACTIVATIONS (the erf or the tanh form of gelu, silu, relu squared), or "xielu":
 act(z) = softplus(p) z^2 + z/2 for z > 0 and (1/2 + softplus(q)) (e^z - 1 - z) + z/2 otherwise, with the layer's two numbers (p, q).
 
 The clamped gated feed-forward: g = min(W_gate xn, L), u = clamp(W_up xn, -L, L), y = W_down (g sigmoid(alpha g) (u + 1)).
@@ -12,10 +12,15 @@ The clamped gated feed-forward: g = min(W_gate xn, L), u = clamp(W_up xn, -L, L)
 The routed feed-forward: a router chooses `top` of E small gated feed-forwards per token (the largest logits; their weights
 the softmax over the chosen logits alone); the weighted sum of their outputs, plus, if there is one, a feed-forward that every
 token uses.  Instead of a router a table [vocab, top] may name the experts of every token id, each weighted 1 / top.  An expert's
-gate is one of the gated epilogues' activations, or "clamped": the clamped gated form above with `limit` and `alpha`."""
+gate is one of the gated epilogues' activations, or "clamped": the clamped gated form above with `limit` and `alpha`.
+
+The scored router (`scored`, a ScoredRouter): scores s = softmax(W_router xn) over ALL experts; the choice goes by s + correction, inside the best
+groups of neighbouring experts; weights s / (sum of the chosen s + 1e-20) * scale.  The last rows of its matrix may be identities, "experts"
+without weights whose output is xn itself."""
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -68,8 +73,8 @@ class DenseMLP(FeedForward):
         """act_params: for "xielu" the layer's two numbers (p, q) as the checkpoint holds them."""
         if w_up.shape != (intermediate, hidden) or w_down.shape != (hidden, intermediate):
             raise ValueError("feed-forward weights do not fit the sizes")
-        if activation not in ops.ACTIVATIONS and activation != "xielu":
-            raise ValueError(f"activation {activation!r} is not one of {sorted(ops.ACTIVATIONS) + ['xielu']}")
+        if activation not in ops.DENSE_ACTIVATIONS and activation != "xielu":
+            raise ValueError(f"activation {activation!r} is not one of {sorted(ops.DENSE_ACTIVATIONS) + ['xielu']}")
         self.hidden, self.intermediate, self.activation = hidden, intermediate, activation
         self.w_up, self.w_down = w_up.contiguous(), w_down.contiguous()
         self.a_pos = self.a_neg = 0.0
@@ -111,6 +116,17 @@ class ClampedGLU(FeedForward):
         ops.linear(act, self.w_down, residual, ops.LINEAR_ACC_F32)
 
 
+@dataclass(frozen=True)
+class ScoredRouter:
+    """How a router's scores become a choice: `groups` equal groups of neighbours of which `keep` take part (1, 1: no groups), the last
+    `identities` outputs without weights of their own, the chosen weights' common factor, and what is added to the scores for the choice alone."""
+    correction: Optional[torch.Tensor] = None       # float32 [experts + identities]
+    groups: int = 1
+    keep: int = 1
+    identities: int = 0
+    scale: float = 1.0
+
+
 class RoutedExperts(FeedForward):
     """w_router float32 [E, hidden] (+ b_router [E]); w_gate_up [E, 2 ff, hidden] (an expert's gate rows, then its up rows) and
     w_down [E, hidden, ff] in the compute dtype; `shared`: a FeedForward every token passes as well (or None).  The router's
@@ -123,33 +139,42 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, hidden: int, intermediate: int, experts: int, top: int, w_router: Optional[torch.Tensor], b_router: Optional[torch.Tensor],
                  w_gate_up: torch.Tensor, w_down: torch.Tensor, shared: Optional[FeedForward] = None, activation: str = "silu",
-                 table: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 1.702):
-        """Either w_router (float32 [E, hidden], with or without b_router) or table (int32 [vocab, >= top]: the experts of every token
+                 table: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 1.702, scored: Optional[ScoredRouter] = None):
+        """With `scored` w_router is [E + identities, hidden] and there is no b_router.  Either w_router (float32 [E, hidden], with or without b_router) or table (int32 [vocab, >= top]: the experts of every token
         id, each weighted 1 / top).  activation: one of the gated epilogues' or "clamped" (with limit and alpha)."""
         E = experts
         if w_gate_up.shape != (E, 2 * intermediate, hidden) or w_down.shape != (E, hidden, intermediate):
             raise ValueError("the experts' weights do not fit the sizes")
         if (w_router is None) == (table is None):
             raise ValueError("the experts are chosen by a router or by a table, one of the two")
-        if w_router is not None and w_router.shape != (E, hidden):
+        outputs = E + (scored.identities if scored is not None else 0)
+        if w_router is not None and w_router.shape != (outputs, hidden):
             raise ValueError("the router does not fit the experts")
+        if scored is not None:
+            if w_router is None or b_router is not None:
+                raise ValueError("a scored router has a matrix and no bias")
+            if scored.groups < 1 or outputs % scored.groups or not 1 <= scored.keep <= scored.groups or top > outputs // scored.groups * scored.keep:
+                raise ValueError("the router's groups do not fit the experts")
+            if scored.correction is not None and scored.correction.shape != (outputs,):
+                raise ValueError("the router's correction does not fit the experts")
         if b_router is not None and (w_router is None or b_router.shape != (E,)):
             raise ValueError("the router's bias does not fit the experts")
         if table is not None and (table.dim() != 2 or table.shape[1] < top or table.dtype != torch.int32):
             raise ValueError("the experts' table is int32 [vocab, top]")
-        if not 1 <= top <= min(E, 32):
+        if not 1 <= top <= min(outputs, 32):
             raise ValueError("a token uses between one and min(experts, 32) experts")
         if activation == "clamped" and not limit > 0:
             raise ValueError("the clamp's limit is positive")
         self.hidden, self.intermediate, self.E, self.top, self.activation, self.shared = hidden, intermediate, E, int(top), activation, shared
-        self.limit, self.alpha = float(limit), float(alpha)
+        self.limit, self.alpha, self.scored = float(limit), float(alpha), scored
+        self.correction = None if scored is None or scored.correction is None else scored.correction.to(torch.float32).contiguous()
         self.w_router = None if w_router is None else w_router.to(torch.float32).contiguous()
         self.b_router = None if b_router is None else b_router.to(torch.float32).contiguous()
         self.table = None if table is None else table.contiguous()
         self.w_gate_up, self.w_down = w_gate_up.contiguous(), w_down.contiguous()
 
     def tensors(self):
-        return [t for t in (self.w_router, self.b_router, self.table, self.w_gate_up, self.w_down) if t is not None] + \
+        return [t for t in (self.w_router, self.b_router, self.correction, self.table, self.w_gate_up, self.w_down) if t is not None] + \
             ([] if self.shared is None else self.shared.tensors())
 
     def weight_bytes(self) -> int:
@@ -164,6 +189,8 @@ class RoutedExperts(FeedForward):
         wts = ws.rows("moe.wts", T, self.top, torch.float32)
         if self.table is not None:
             ops.experts_route_table(ctx.tokens, self.table, self.E, self.top, ids, wts)
+        elif self.scored is not None:
+            ops.experts_route_scored(xn, self.w_router, self.correction, self.top, self.scored.groups, self.scored.keep, self.scored.scale, ids, wts)
         else:
             ops.experts_route(xn, self.w_router, self.b_router, self.top, ids, wts)
         if T * self.top >= self.GROUPED_FROM and ops.experts_grouped_takes(xn, self.w_gate_up, self.w_down):

@@ -35,6 +35,9 @@ def _register_builtin() -> None:
     from .block import OutputNormBlock, PreNormBlock, SandwichNormBlock
     from .gla import GatedLinearAttention
     from .mixed_attention import MixedHeadAttention
+    from .parallel import ParallelMixer
+    from .rotary_attention import RotaryAttention
+    from .ssd import StateSpaceMixer
     from .diff_attention import DiffAttention
     from .mlstm import MatrixLSTM
     from .delta import ChannelDeltaRule, GatedDeltaRule
@@ -51,6 +54,9 @@ def _register_builtin() -> None:
     register_part("mixer", "mlstm", MatrixLSTM)
     register_part("mixer", "gla", GatedLinearAttention)
     register_part("mixer", "mixed_attention", MixedHeadAttention)
+    register_part("mixer", "rotary_attention", RotaryAttention)
+    register_part("mixer", "ssd", StateSpaceMixer)
+    register_part("mixer", "parallel", ParallelMixer)
     register_part("feed_forward", "clamped_glu", ClampedGLU)
     register_part("feed_forward", "routed_experts", RoutedExperts)
     register_part("feed_forward", "swiglu", SwiGLU)
