@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, as one JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
-                    [--model 135M|360M|1.7B] [--workload decode|mixed|prefill8k|lupanex|siparax|manatar|tinevik]
+                    [--model 135M|360M|1.7B] [--workload decode|mixed|prefill8k|lupanex|siparax|manatar|tinevik|lirutar]
 
 The default run is SmolLM2-135M's sizes with random weights (N(0, 0.02), norm weights 1, seed 0) in
 bfloat16, a batch of 8 requests each decoding from its own 2,048-token random prompt, cache context
@@ -541,9 +541,11 @@ def kind_of(launch):
         return "mlstm"
     if launch.startswith("gla"):
         return "gla"
+    if launch.startswith("ssd"):
+        return "ssd"
     if launch == "latent_expand_gate":
         return "expand"
-    if launch in ("sandwich_step", "xielu", "mixed_attn_prepare", "embed_scaled"):
+    if launch in ("sandwich_step", "xielu", "mixed_attn_prepare", "embed_scaled", "pass_input"):
         return "between"
     if launch in ("embed_hashed", "residual_norm_step", "glu_clamped", "diff_attn_prepare", "diff_attn_combine"):
         return "between"
@@ -857,6 +859,79 @@ def tinevik_run(a, pk, clocks):
     return results
 
 
+# ---------------------------------------------------------------------------------------------------------------
+# --workload lirutar
+# ---------------------------------------------------------------------------------------------------------------
+
+# Lirutar beside Tinevik, the engine's closest design: a recurrent matrix state, an attention over a window with values of their own size,
+# clamped experts on the same grouped products.  Equal width, runs of a layer (six layers of which two run twice: eight), attention heads and
+# sizes, size of the recurrent state a layer, and weights a token uses in the feed-forwards (2 of 8 experts a quarter as wide and a shared one
+# half as wide, against Tinevik's 2 of 8 half as wide; the first layer dense).  Tinevik's layers have ONE mixer each (a recurrent one six
+# times, an attention twice); every layer of Lirutar has both, so it does four times the attention's work.
+LIRUTAR_SIZES = {
+    "w1024": dict(TINEVIK_SIZES["w1024"], ssd=dict(heads=16, vdim=64, state=64, groups=4)),
+    "w2048": dict(TINEVIK_SIZES["w2048"], ssd=dict(heads=32, vdim=64, state=128, groups=8)),
+}
+LIRUTAR_LOOP = dict(start=1, stop=3, times=2)
+LIRUTAR_EXPERTS, LIRUTAR_IDENTITIES, LIRUTAR_TOP = 8, 2, 2
+
+
+def lirutar_config(sz):
+    dk, dv, r = sz["dim"], sz["vdim"], sz["ssd"]
+    left = dict(heads=2 * sz["heads"], kv_heads=sz["kv"], dim=dk, vdim=dv, scale=dk ** -0.5, rot=dict(base=100000.0, dims=dk // 2), mask=dict(size=sz["window"]))
+    right = dict(heads=r["heads"], vdim=r["vdim"], state=r["state"], groups=r["groups"], conv=4, norm_groups=r["groups"])
+    mixer = dict(left=left, right=right, left_scale=0.7, right_scale=0.8)
+    moe = dict(kind="moe", expert=dict(ff=sz["ff"] // 4, limit=7.0), shared=dict(ff=sz["ff"] // 2, limit=7.0),
+               router=dict(experts=LIRUTAR_EXPERTS, identity=LIRUTAR_IDENTITIES, top=LIRUTAR_TOP, groups=dict(count=5, keep=3), scale=2.0))
+    n = sz["layers"] - (LIRUTAR_LOOP["stop"] - LIRUTAR_LOOP["start"]) * (LIRUTAR_LOOP["times"] - 1)
+    layers = [dict(type="parallel", mixer=mixer, mlp=dict(kind="dense", ff=3 * sz["ff"] // 2) if i == 0 else moe) for i in range(n)]
+    return dict(architecture="Lirutar", vocab=LUPANEX_VOCAB, width=sz["width"], norm=dict(eps=1e-6), loop=LIRUTAR_LOOP, layers=layers)
+
+
+def lirutar_work(sz, T):
+    """Algorithmic work of one T-token prompt, by kind of kernel: (flops, bytes)."""
+    W, L, r = sz["width"], sz["layers"], sz["ssd"]
+    H, G, dk, dv, win = 2 * sz["heads"], sz["kv"], sz["dim"], sz["vdim"], sz["window"]
+    inner, chan = r["heads"] * r["vdim"], r["heads"] * r["vdim"] + 2 * r["groups"] * r["state"]
+    att_rows, ssd_rows = H * dk + G * dk + G * dv, inner + chan + r["heads"]
+    seen = float(T) * (T + 1) / 2 if win >= T else float(T) * win - win * (win - 1) / 2.0        # (query, key) pairs inside the window
+    e_ff, used = sz["ff"] // 4, LIRUTAR_TOP * LIRUTAR_EXPERTS / (LIRUTAR_EXPERTS + LIRUTAR_IDENTITIES)      # a token's pairs that are experts
+    return {
+        "product": (2.0 * T * (L * W * (att_rows + ssd_rows + H * dv + inner) + LIRUTAR_LOOP["times"] * 2 * W * W + (L - 1) * 3 * W * (sz["ff"] // 2)
+                               + 2 * W * (3 * sz["ff"] // 2)), 0.0),
+        "attention": (L * 2.0 * seen * H * (dk + dv), 0.0),
+        "ssd": (L * 5.0 * T * inner * r["state"], L * T * (4.0 * ssd_rows + 2.0 * inner)),
+        "experts": ((L - 1) * 2.0 * T * used * 3 * W * e_ff, (L - 1) * LIRUTAR_EXPERTS * 3.0 * W * e_ff * 2),
+        "between": (0.0, (2 * L + 1) * T * W * 6.0 + L * T * 6.0 * att_rows + (L - 1) * T * (sz["ff"] // 2) * 6.0 + (LIRUTAR_LOOP["times"] + 1) * T * W * 6.0),
+    }
+
+
+def lirutar_run(a, pk, clocks):
+    import torch
+    from vitna_anchor_b200.engine.loading import random_model_on_device
+    results = {}
+    for name, sz in LIRUTAR_SIZES.items():
+        row = {}
+        for which, cfg, work in (("lirutar", lirutar_config(sz), lirutar_work(sz, PREFILL_TOKENS)),
+                                 ("tinevik", tinevik_config(TINEVIK_SIZES[name]), tinevik_work(TINEVIK_SIZES[name], PREFILL_TOKENS))):
+            model = random_model_on_device(cfg, 0)
+            if model.max_positions > CONTEXT:
+                model.max_positions = CONTEXT           # the design has no limit of its own; the run's cache has
+            pf = prefill_run(model, None, clocks, repeats=3)
+            dec = decode_run(model, a.batch, min(a.steps, 32), a.warmup, clocks, with_e2e=False)
+            flops = sum(f for f, _ in work.values())
+            row[which] = {"weights_mb": round(model.step_weight_bytes() / 1e6, 1),
+                          "prefill_2048": {"tokens_per_s": round(pf["value"]), "ms": round(pf["ms"], 3),
+                                           "frac_bf16": round(flops / (pf["ms"] * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)},
+                          f"decode_b{a.batch}": {"tokens_per_s": round(dec["value"]), "ms_per_step": round(dec["ms_per_step"], 4),
+                                                 "frac_hbm": round(dec["gbs"] / pk["hbm_gbs"], 4), "launches_per_step": dec["launches"] // min(a.steps, 32)},
+                          "prompt_by_kind": prompt_by_kind(model, work, pk)}
+            del model
+            torch.cuda.empty_cache()
+        results[name] = row
+    return results
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -865,10 +940,10 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--model", default="135M", choices=sorted(MODELS), help="layer sizes: SmolLM2-135M (the default), 360M or 1.7B")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "prefill8k", "lupanex", "siparax", "manatar", "tinevik"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "prefill8k", "lupanex", "siparax", "manatar", "tinevik", "lirutar"],
                     help="decode (the default line), mixed (32 requests, 512-token portions beside decodes), prefill8k, lupanex "
                          "(the Lupanex design beside a Llama model of equal size), siparax and manatar (those designs beside Lupanex), "
-                         "tinevik (that design beside Manatar with routed feed-forwards)")
+                         "tinevik (that design beside Manatar with routed feed-forwards), lirutar (that design beside Tinevik)")
     ap.add_argument("--no-points", action="store_true", help="skip the other batches, models and the prefill")
     ap.add_argument("--only-prefill", action="store_true", help="run the prefill measurement alone (for profiling)")
     ap.add_argument("--profile-region", default="", choices=["", "decode", "prefill"],
@@ -927,6 +1002,15 @@ def main():
         r = tinevik_run(a, pk, clocks)
         clocks.stop()
         print(json.dumps({"metric": "Tinevik beside Manatar with routed feed-forwards at equal width, depth, heads and weights a token uses: tokens/s "
+                          f"of a 2,048-token prompt and of batch-{a.batch} decoding from 2,048-token prompts; a prompt's time by kind of kernel "
+                          "against its roofline", "impl": "ours", "dtype": "bf16",
+                          "data": "synthetic: random weights drawn on the device, uniform-random token ids", "peaks": pk, "sizes": r,
+                          "clocks": clocks.summary()}))
+        return 0
+    if a.workload == "lirutar":
+        r = lirutar_run(a, pk, clocks)
+        clocks.stop()
+        print(json.dumps({"metric": "Lirutar beside Tinevik at equal width, runs of a layer, heads and feed-forward weights a token uses: tokens/s "
                           f"of a 2,048-token prompt and of batch-{a.batch} decoding from 2,048-token prompts; a prompt's time by kind of kernel "
                           "against its roofline", "impl": "ours", "dtype": "bf16",
                           "data": "synthetic: random weights drawn on the device, uniform-random token ids", "peaks": pk, "sizes": r,
