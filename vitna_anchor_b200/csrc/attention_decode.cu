@@ -317,6 +317,11 @@ int launch_decode_mma(const void* q, const void* cache, const int32_t* bt, const
                       int hd, int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
                       cudaStream_t stream);
 
+int launch_decode_mma_values(const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
+                             const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
+                             int hd, int vd, int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
+                             int out_ld, int v_in_key, int v_share, cudaStream_t stream);
+
 // attention_decode_tma.cu: the persistent kernel for large launches (bfloat16, head size 64).
 bool decode_tma_takes(int n_tokens, int nh, int nkv, int hd, int page_size, int pages, int grid_splits, const void* q, const void* cache,
                       const int* error);
@@ -425,6 +430,10 @@ VK_API int vk_attention_decode_biased(const void* q, const void* cache, const in
     float* part_o = (float*)base;
     float* part_ml = (float*)(base + up((size_t)scratch_tokens * nh * splits * wide * 4));
     int* counters = (int*)((char*)part_ml + up((size_t)scratch_tokens * nh * splits * 2 * 4));
+    auto built = [](int n) { return n == 32 || n == 64 || n == 96 || n == 128; };
+    if (dtype == 1 && !dist_bias && built(hd) && built(vd) && ((uintptr_t)q % 16 == 0) && scale > 0.0f)
+        return launch_decode_mma_values(q, cache, block_tables, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, hd,
+                                        vd, page_size, max_blocks, splits, grid_splits, tiles, scale, window, out_ld, v_in_key, v_share, stream);
     const size_t smem_base = (size_t)(DEC_G_TILE * hd + DEC_G_TILE * DEC_SPLIT + DEC_THREADS * vec) * sizeof(float);
     const size_t smem_async = smem_base + (size_t)DEC_SPLIT * (hd + vd + 2 * vec) * (dtype == 0 ? 4 : 2);
     const bool async = smem_async <= 100 * 1024;        // two blocks a multiprocessor

@@ -21,7 +21,10 @@
 // transposed in registers (movmatrix) on their way into the 8-column operand.  Half the products and
 // exponentials; the parts that the warp leaves have the same layout either way.
 //
-// Instantiated for head sizes 16, 32, 64, 96 and 128; attention_decode.cu takes the others and float32.
+// Values may have another size than the keys (VD; a page is then [nkv][page_size][HD] keys followed by [nkv / v_share][page_size][VD] values,
+// v_share neighbouring key heads reading one value head), or be the first VD values of the keys (v_in_key; a page then holds the keys
+// alone), and the rows of the output may lie apart (out_ld).  Instantiated for head sizes 16, 32, 64, 96 and 128, and for every pair of key and
+// value sizes of 32, 64, 96 and 128; attention_decode.cu takes the others and float32.
 #include "common.cuh"
 
 namespace vk {
@@ -66,6 +69,8 @@ struct DmArgs {
     int nh, nkv, page_size, page_shift, max_blocks, max_splits, counter_tiles;   // page_shift: log2 of page_size, or -1
     float scale;
     int window;
+    int out_ld;                             // elements between rows of out
+    int v_in_key, v_share;
 };
 
 __device__ __forceinline__ DmItem dm_item(const DmArgs& a, int zi, int y, int split) {
@@ -113,54 +118,80 @@ __device__ __forceinline__ uint32_t dm_pack(float x, float y) {
 // The key and value at the token's own position are left out: they are what the kernel before this one writes, and
 // this copy runs before the wait for that kernel (dm_copy_own brings them afterwards).  Every earlier key of the
 // request was written by an earlier step.  Returns the page of the token's own position (to every lane).
-template <int HD>
+template <int HD, int VD>
 __device__ __forceinline__ int dm_copy_warp(const DmArgs& a, const DmItem& it, __nv_bfloat16* sk, __nv_bfloat16* sv) {
     typedef __nv_bfloat16 T;
-    constexpr int LD = HD + 8, CH = HD / 8;             // CH pieces of 16 bytes a row
+    constexpr int LD = HD + 8, LDV = VD + 8, CH = HD / 8, CHV = VD / 8;     // pieces of 16 bytes a row
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const size_t page_stride = (size_t)2 * a.nkv * a.page_size * HD;
-    const size_t v_off = (size_t)a.nkv * a.page_size * HD;
+    const size_t page_stride = (size_t)a.page_size * (a.v_in_key ? a.nkv * HD : a.nkv * HD + a.nkv / a.v_share * VD);
+    const size_t v_off = a.v_in_key ? 0 : (size_t)a.nkv * a.page_size * HD;
+    const int v_ld = a.v_in_key ? HD : VD, vh = it.kvh / a.v_share;
     const int wk0 = it.k0 + warp * 32;                  // the warp's first key
     const int pg0 = a.page_shift >= 0 ? wk0 >> a.page_shift : wk0 / a.page_size;
     const int pg_last = a.page_shift >= 0 ? it.pos >> a.page_shift : it.pos / a.page_size;     // the request has pages up to here
     const int my_page = pg0 + lane <= pg_last ? it.bt[pg0 + lane] : 0;        // at most 32 pages hold 32 keys
-#pragma unroll
-    for (int i = 0; i < CH; i++) {
-        const int c = i * 32 + lane;
-        const int kl = warp * 32 + c / CH, part = c % CH;
+    // piece `part` of key kl: its place among the pages' keys (which = 0) or values (1)
+    auto one = [&](int c, int ch, int which) {
+        const int kl = warp * 32 + c / ch, part = c % ch;
         const int key = it.k0 + kl;
         const int pg = a.page_shift >= 0 ? key >> a.page_shift : key / a.page_size;
         const int page = __shfl_sync(0xffffffffu, my_page, pg - pg0);
-        T* dk = sk + kl * LD + part * 8;
-        T* dv = sv + kl * LD + part * 8;
+        const int off = key - pg * a.page_size;
+        const T* src = a.cache + (size_t)page * page_stride + part * 8 +
+                       (which ? v_off + ((size_t)vh * a.page_size + off) * v_ld : ((size_t)it.kvh * a.page_size + off) * HD);
+        T* dst = which ? sv + kl * LDV + part * 8 : sk + kl * LD + part * 8;
         if (kl < it.nkeys && key >= it.lo) {
-            if (key < it.pos) {
-                const int off = key - pg * a.page_size;
-                const T* kr = a.cache + (size_t)page * page_stride + ((size_t)it.kvh * a.page_size + off) * HD + part * 8;
-                dm_cp_async16(dk, kr);
-                dm_cp_async16(dv, kr + v_off);
-            }
+            if (key < it.pos) dm_cp_async16(dst, src);
         } else {
-            *reinterpret_cast<uint4*>(dk) = make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(dv) = make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
+    };
+    if (HD == VD && !a.v_in_key && a.v_share == 1) {
+#pragma unroll
+        for (int i = 0; i < CH; i++) {
+            const int c = i * 32 + lane;
+            const int kl = warp * 32 + c / CH, part = c % CH;
+            const int key = it.k0 + kl;
+            const int pg = a.page_shift >= 0 ? key >> a.page_shift : key / a.page_size;
+            const int page = __shfl_sync(0xffffffffu, my_page, pg - pg0);
+            T* dk = sk + kl * LD + part * 8;
+            T* dv = sv + kl * LD + part * 8;
+            if (kl < it.nkeys && key >= it.lo) {
+                if (key < it.pos) {
+                    const int off = key - pg * a.page_size;
+                    const T* kr = a.cache + (size_t)page * page_stride + ((size_t)it.kvh * a.page_size + off) * HD + part * 8;
+                    dm_cp_async16(dk, kr);
+                    dm_cp_async16(dv, kr + v_off);
+                }
+            } else {
+                *reinterpret_cast<uint4*>(dk) = make_uint4(0, 0, 0, 0);
+                *reinterpret_cast<uint4*>(dv) = make_uint4(0, 0, 0, 0);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < CH; i++) one(i * 32 + lane, CH, 0);
+#pragma unroll
+        for (int i = 0; i < CHV; i++) one(i * 32 + lane, CHV, 1);
     }
     return __shfl_sync(0xffffffffu, my_page, min(max(pg_last - pg0, 0), 31));
 }
 
-// The key and value at the token's own position, for the warp whose 32 keys hold it: lanes 0 .. HD/8-1 copy a piece each.
-template <int HD>
+// The key and value at the token's own position, for the warp whose 32 keys hold it: lanes 0 .. HD/8-1 (VD/8-1) copy a piece each.
+template <int HD, int VD>
 __device__ __forceinline__ void dm_copy_own(const DmArgs& a, const DmItem& it, int own_page, __nv_bfloat16* sk, __nv_bfloat16* sv) {
     typedef __nv_bfloat16 T;
-    constexpr int LD = HD + 8, CH = HD / 8;
+    constexpr int LD = HD + 8, LDV = VD + 8;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int kl = it.pos - it.k0;
-    if (kl < warp * 32 || kl >= warp * 32 + 32 || lane >= CH) return;
+    if (kl < warp * 32 || kl >= warp * 32 + 32) return;
     const int pg = a.page_shift >= 0 ? it.pos >> a.page_shift : it.pos / a.page_size;
     const int off = it.pos - pg * a.page_size;
-    const T* kr = a.cache + (size_t)own_page * 2 * a.nkv * a.page_size * HD + ((size_t)it.kvh * a.page_size + off) * HD + lane * 8;
-    dm_cp_async16(sk + kl * LD + lane * 8, kr);
-    dm_cp_async16(sv + kl * LD + lane * 8, kr + (size_t)a.nkv * a.page_size * HD);
+    const T* page = a.cache + (size_t)own_page * a.page_size * (a.v_in_key ? a.nkv * HD : a.nkv * HD + a.nkv / a.v_share * VD);
+    const T* kr = page + ((size_t)it.kvh * a.page_size + off) * HD;
+    const T* vr = a.v_in_key ? kr : page + (size_t)a.nkv * a.page_size * HD + ((size_t)(it.kvh / a.v_share) * a.page_size + off) * VD;
+    if (lane < HD / 8) dm_cp_async16(sk + kl * LD + lane * 8, kr + lane * 8);
+    if (lane < VD / 8) dm_cp_async16(sv + kl * LDV + lane * 8, vr + lane * 8);
 }
 
 // The queries of the item's heads as the 16-row operand of m16n8k16, straight from global memory into registers
@@ -191,12 +222,12 @@ __device__ __forceinline__ uint32_t dm_movmatrix_trans(uint32_t x) {
 // 8-column operand) and O^T[16 dims x 8 heads] = V^T P^T (V^T by a transposing ldmatrix; the probabilities go from
 // the score registers through movmatrix into the 8-column operand, again as a high and a low bfloat16 part).  Half the
 // products and half the exponentials of the routine with the heads as rows, which wastes thirteen of sixteen rows on
-// a group of three heads.  Leaves the warp's maxima and sums in wml and its unnormalised output [head][HD] in wo.
-template <int HD>
+// a group of three heads.  Leaves the warp's maxima and sums in wml and its unnormalised output [head][VD] in wo.
+template <int HD, int VD>
 __device__ __forceinline__ void dm_warp_few_heads(const DmArgs& a, const DmItem& it, const __nv_bfloat16* sk, const __nv_bfloat16* sv,
                                                   float* wml, float* wo, float scale_log2) {
     typedef __nv_bfloat16 T;
-    constexpr int LD = HD + 8, KSTEPS = HD / 16, HB = HD / 16;
+    constexpr int LD = HD + 8, LDV = VD + 8, KSTEPS = HD / 16, HB = VD / 16;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gq = lane >> 2, qd = lane & 3;
     const int wk0 = it.k0 + warp * 32, pos = it.pos, lo = it.lo, gt = it.gt;
     // the queries as the 8-column operand: lane (gq, qd) holds head gq, dims 2qd, 2qd+1 and +8 of each k-step
@@ -282,7 +313,7 @@ __device__ __forceinline__ void dm_warp_few_heads(const DmArgs& a, const DmItem&
         for (int hb = 0; hb < HB; hb++) {
             uint32_t af[4];
             dm_ldsm_x4_trans(af[0], af[1], af[2], af[3],
-                             sv + (warp * 32 + kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * LD + hb * 16 + ((lane >> 3) & 1) * 8);
+                             sv + (warp * 32 + kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * LDV + hb * 16 + ((lane >> 3) & 1) * 8);
             dm_mma(o[hb], af, ph[kb][0], ph[kb][1]);
             dm_mma(o[hb], af, pl[kb][0], pl[kb][1]);
         }
@@ -295,18 +326,18 @@ __device__ __forceinline__ void dm_warp_few_heads(const DmArgs& a, const DmItem&
         for (int e = 0; e < 2; e++) {
             const int head = 2 * qd + e;
             if (head < gt) {
-                wo[head * HD + d] = o[hb][e];
-                wo[head * HD + d + 8] = o[hb][2 + e];
+                wo[head * VD + d] = o[hb][e];
+                wo[head * VD + d + 8] = o[hb][2 + e];
             }
         }
     }
 }
 
-// Shared memory of a block: keys [256][HD+8], values [256][HD+8] and the warps' maxima and sums [8][16][2].  A warp's unnormalised output [16][HD] float32 lies over its own 32 keys,
-// dead once it has its scores.  74 KB at HD = 64: three blocks a multiprocessor.
-template <int HD> struct DmSmem {
-    static constexpr int LD = HD + 8;
-    static constexpr size_t KV_BYTES = (size_t)2 * DM_SPLIT * LD * 2;
+// Shared memory of a block: keys [256][HD+8], values [256][VD+8] and the warps' maxima and sums [8][16][2].  A warp's unnormalised output
+// [16][VD] float32 lies over its own 32 keys (values, where those are longer), dead once it has its scores (its sums).  74 KB at HD = VD = 64:
+// three blocks a multiprocessor.
+template <int HD, int VD> struct DmSmem {
+    static constexpr size_t KV_BYTES = (size_t)DM_SPLIT * (HD + VD + 16) * 2;
     static constexpr size_t BYTES = KV_BYTES + 8 * DM_ROWS * 2 * 4;
 };
 
@@ -314,14 +345,14 @@ template <int HD> struct DmSmem {
 // probabilities going from the score registers straight into the 16-row operand (as a high and a low bfloat16
 // part, p = hi + lo to about 2^-17).  Only then do the warps meet: their eight parts are weighted and added in
 // warp order, and the block leaves its partial (or, for a single split, the result).
-template <int HD>
-__global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode_mma_kernel(const DmArgs a) {
+template <int HD, int VD>
+__global__ void __launch_bounds__(DM_THREADS, HD + VD <= 128 ? 3 : 1) attention_decode_mma_kernel(const DmArgs a) {
     typedef __nv_bfloat16 T;
-    typedef DmSmem<HD> L;
-    constexpr int LD = HD + 8, KSTEPS = HD / 16, DBLK = HD / 8;
+    typedef DmSmem<HD, VD> L;
+    constexpr int LD = HD + 8, LDV = VD + 8, KSTEPS = HD / 16, DBLK = VD / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     T* sk = reinterpret_cast<T*>(smem_raw);                 // [256][LD]
-    T* sv = sk + DM_SPLIT * LD;                             // [256][LD]
+    T* sv = sk + DM_SPLIT * LD;                             // [256][LDV]
     float* wml = reinterpret_cast<float*>(smem_raw + L::KV_BYTES);   // [8 warps][16 rows][2]: maximum, sum
     __shared__ int is_last;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -339,17 +370,20 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
     // The keys and values of earlier steps are asked for before the wait: they are most of what a block reads,
     // and the kernel before this one writes the token's own key and value only.
     int own_page = 0;
-    if (warp_on) own_page = dm_copy_warp<HD>(a, it, sk, sv);
+    if (warp_on) own_page = dm_copy_warp<HD, VD>(a, it, sk, sv);
     dependency_wait();                          // q and the token's own key and value come from the kernel before this one
     let_dependents_start();
 
-    float* wo = reinterpret_cast<float*>(sk + warp * 32 * LD);       // [16][HD], over the warp's own keys
+    constexpr bool OVER_K = VD <= HD;
+    constexpr int WO_LD = OVER_K ? LD : LDV;
+    T* wo_base = OVER_K ? sk : sv;
+    float* wo = reinterpret_cast<float*>(wo_base + warp * 32 * WO_LD);       // [16][VD], over the warp's own keys or values
     if (warp_on && gt <= 8) {
-        dm_copy_own<HD>(a, it, own_page, sk, sv);
+        dm_copy_own<HD, VD>(a, it, own_page, sk, sv);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        dm_warp_few_heads<HD>(a, it, sk, sv, wml, wo, scale_log2);
+        dm_warp_few_heads<HD, VD>(a, it, sk, sv, wml, wo, scale_log2);
     } else if (warp_on) {
-        dm_copy_own<HD>(a, it, own_page, sk, sv);
+        dm_copy_own<HD, VD>(a, it, own_page, sk, sv);
         asm volatile("cp.async.commit_group;" ::: "memory");
         uint32_t qf[KSTEPS][4];
         dm_load_q<HD>(a, it, qf);
@@ -426,7 +460,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
 #pragma unroll
             for (int db = 0; db < DBLK; db += 2) {
                 uint32_t b0, b1, b2, b3;
-                dm_ldsm_x4_trans(b0, b1, b2, b3, sv + (warp * 32 + kk * 16 + (lane & 15)) * LD + (db + (lane >> 4)) * 8);
+                dm_ldsm_x4_trans(b0, b1, b2, b3, sv + (warp * 32 + kk * 16 + (lane & 15)) * LDV + (db + (lane >> 4)) * 8);
                 dm_mma(o[db], ph[kk], b0, b1);
                 dm_mma(o[db], pl[kk], b0, b1);
                 dm_mma(o[db + 1], ph[kk], b2, b3);
@@ -437,8 +471,8 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
 #pragma unroll
         for (int db = 0; db < DBLK; db++) {
             const int d = db * 8 + qd * 2;
-            if (gq < gt) *reinterpret_cast<float2*>(wo + gq * HD + d) = make_float2(o[db][0], o[db][1]);
-            if (gq + 8 < gt) *reinterpret_cast<float2*>(wo + (gq + 8) * HD + d) = make_float2(o[db][2], o[db][3]);
+            if (gq < gt) *reinterpret_cast<float2*>(wo + gq * VD + d) = make_float2(o[db][0], o[db][1]);
+            if (gq + 8 < gt) *reinterpret_cast<float2*>(wo + (gq + 8) * VD + d) = make_float2(o[db][2], o[db][3]);
         }
     } else if (lane < DM_ROWS) {
         *reinterpret_cast<float2*>(wml + (warp * DM_ROWS + lane) * 2) = make_float2(-INFINITY, 0.0f);
@@ -449,8 +483,8 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
     // order (row maximum, weights exp(own maximum - row maximum), sum); the threads of a row's first column also
     // leave the row's maximum and sum
     const bool single = n_active == 1;
-    for (int i = tid; i < gt * HD; i += DM_THREADS) {
-        const int row = i / HD, d = i % HD;
+    for (int i = tid; i < gt * VD; i += DM_THREADS) {
+        const int row = i / VD, d = i % VD;
         float2 ml[8];
 #pragma unroll
         for (int w = 0; w < 8; w++) ml[w] = *reinterpret_cast<const float2*>(wml + (w * DM_ROWS + row) * 2);
@@ -463,12 +497,12 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
             if (ml[w].x == -INFINITY) continue;     // a warp without a counted key left nothing
             const float e = dm_ex2(ml[w].x - m);
             l += ml[w].y * e;
-            acc += reinterpret_cast<const float*>(sk + w * 32 * LD)[row * HD + d] * e;
+            acc += reinterpret_cast<const float*>(wo_base + w * 32 * WO_LD)[row * VD + d] * e;
         }
         if (single) {
-            a.out[((size_t)t * nh + h0 + row) * HD + d] = __float2bfloat16_rn(acc / l);
+            a.out[(size_t)t * a.out_ld + (h0 + row) * VD + d] = __float2bfloat16_rn(acc / l);
         } else {
-            a.part_o[(((size_t)zi * nh + h0 + row) * max_splits + split) * HD + d] = acc;
+            a.part_o[(((size_t)zi * nh + h0 + row) * max_splits + split) * VD + d] = acc;
             if (d == 0) *reinterpret_cast<float2*>(a.part_ml + (((size_t)zi * nh + h0 + row) * max_splits + split) * 2) = make_float2(m, l);
         }
     }
@@ -492,10 +526,10 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
     // trip), and folded into a running maximum, sum and output in split order (the same order whatever else is in
     // the batch).
     constexpr int TRIP = 16;
-    for (int i = tid; i < gt * HD; i += DM_THREADS) {
-        const int h = i / HD, d = i % HD;
+    for (int i = tid; i < gt * VD; i += DM_THREADS) {
+        const int h = i / VD, d = i % VD;
         const float2* ml = reinterpret_cast<const float2*>(a.part_ml) + ((size_t)zi * nh + h0 + h) * max_splits + first_split;
-        const float* po = a.part_o + (((size_t)zi * nh + h0 + h) * max_splits + first_split) * HD + d;
+        const float* po = a.part_o + (((size_t)zi * nh + h0 + h) * max_splits + first_split) * VD + d;
         float mm = -INFINITY, l = 0.0f, o = 0.0f;
         for (int j0 = 0; j0 < n_active; j0 += TRIP) {
             float2 st[TRIP];
@@ -504,7 +538,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
             for (int j = 0; j < TRIP; j++) {
                 const bool on = j0 + j < n_active;
                 st[j] = on ? __ldcg(ml + j0 + j) : make_float2(-INFINITY, 0.0f);
-                pv[j] = on ? __ldcg(po + (size_t)(j0 + j) * HD) : 0.0f;
+                pv[j] = on ? __ldcg(po + (size_t)(j0 + j) * VD) : 0.0f;
             }
             float cm = mm;
 #pragma unroll
@@ -520,27 +554,27 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 3 : 1) attention_decode
             }
             mm = cm;
         }
-        a.out[((size_t)t * nh + h0 + h) * HD + d] = __float2bfloat16_rn(o / l);
+        a.out[(size_t)t * a.out_ld + (h0 + h) * VD + d] = __float2bfloat16_rn(o / l);
     }
 }
 
-template <int HD>
+template <int HD, int VD>
 static int launch_dm(const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
                      const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
                      int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
-                     cudaStream_t stream) {
+                     int out_ld, int v_in_key, int v_share, cudaStream_t stream) {
     const int g = nh / nkv, tiles = nkv * ((g + DM_ROWS - 1) / DM_ROWS);
     int shift = -1;
     for (int b = 0; b < 30; b++) if ((1 << b) == page_size) shift = b;
     DmArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, token_seg, positions, tok_list, (__nv_bfloat16*)out, part_o,
-             part_ml, counters, nh, nkv, page_size, shift, max_blocks, splits, counter_tiles, scale, window};
+             part_ml, counters, nh, nkv, page_size, shift, max_blocks, splits, counter_tiles, scale, window, out_ld, v_in_key, v_share};
     // Three blocks a multiprocessor pay when there are several waves of blocks; with a single wave (a small batch)
     // two blocks and a larger first-level cache were measured faster, so the small launch asks for more shared
     // memory than it uses.
     const long long blocks = (long long)n_tokens * tiles * grid_splits;
-    size_t smem = DmSmem<HD>::BYTES;
+    size_t smem = DmSmem<HD, VD>::BYTES;
     if (blocks < 3 * 148 * 2 && smem < 100 * 1024) smem = 100 * 1024;
-    auto kern = attention_decode_mma_kernel<HD>;
+    auto kern = attention_decode_mma_kernel<HD, VD>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
@@ -554,10 +588,46 @@ int launch_decode_mma(const void* q, const void* cache, const int32_t* bt, const
                       int hd, int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
                       cudaStream_t stream) {
 #define GO(HD)                                                                                                                   \
-    return launch_dm<HD>(q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
-                         max_blocks, splits, grid_splits, counter_tiles, scale, window, stream)
+    return launch_dm<HD, HD>(q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
+                         max_blocks, splits, grid_splits, counter_tiles, scale, window, nh * HD, 0, 1, stream)
     switch (hd) {
         case 16: GO(16);
+        case 32: GO(32);
+        case 64: GO(64);
+        case 96: GO(96);
+        case 128: GO(128);
+    }
+#undef GO
+    return VK_BAD_SHAPE;
+}
+
+template <int HD>
+static int launch_dm_values(int vd, const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
+                            const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
+                            int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window, int out_ld,
+                            int v_in_key, int v_share, cudaStream_t stream) {
+#define GO(VD)                                                                                                                        \
+    return launch_dm<HD, VD>(q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
+                             max_blocks, splits, grid_splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, stream)
+    switch (vd) {
+        case 32: GO(32);
+        case 64: GO(64);
+        case 96: GO(96);
+        case 128: GO(128);
+    }
+#undef GO
+    return VK_BAD_SHAPE;
+}
+
+// Values of their own size and output rows that lie apart, key and value sizes of 32, 64, 96 and 128 (called by vk_attention_decode_biased).
+int launch_decode_mma_values(const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
+                             const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
+                             int hd, int vd, int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
+                             int out_ld, int v_in_key, int v_share, cudaStream_t stream) {
+#define GO(HD)                                                                                                                             \
+    return launch_dm_values<HD>(vd, q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
+                                max_blocks, splits, grid_splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, stream)
+    switch (hd) {
         case 32: GO(32);
         case 64: GO(64);
         case 96: GO(96);

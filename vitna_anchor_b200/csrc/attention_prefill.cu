@@ -56,11 +56,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// Two blocks a multiprocessor where their shared memory lets them; else one, with all its registers.
+constexpr int pf_blocks(int hd, int vd) { return (PF_BM * (hd + 8) + 4 * PF_BN * (hd + vd + 16)) * 2 + 2048 <= 113 * 1024 ? 2 : 1; }
+
 template <int HD, int VD>
-__global__ void __launch_bounds__(PF_THREADS, 2) attention_prefill_kernel(
+__global__ void __launch_bounds__(PF_THREADS, pf_blocks(HD, VD)) attention_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache, const int32_t* __restrict__ block_tables,
     const int32_t* __restrict__ tiles, __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int max_blocks, float scale,
-    int window, const float* __restrict__ dist_bias, int max_dist, int v_in_key, int v_share, int out_ld) {
+    int window, const float* __restrict__ dist_bias, int max_dist, int v_in_key, int v_share, int out_ld, int page_shift) {
     typedef __nv_bfloat16 T;
     constexpr int LD = HD + 8;                      // padded row: 16-byte shifts keep ldmatrix free of bank conflicts
     constexpr int LDV = VD + 8;
@@ -108,15 +111,16 @@ __global__ void __launch_bounds__(PF_THREADS, 2) attention_prefill_kernel(
     auto load_kv = [&](int kt, int buf) {
         T* dk = sk + buf * PF_BN * LD;
         T* dv = sv + buf * PF_BN * LDV;
+#pragma unroll 4
         for (int i = tid; i < PF_BN * (CHUNKS + CHUNKS_V); i += PF_GROUP) {
             const int r = i / (CHUNKS + CHUNKS_V), c = i % (CHUNKS + CHUNKS_V);
             const int key = kt * PF_BN + r;
             T* dst = c < CHUNKS ? dk + r * LD + c * 8 : dv + r * LDV + (c - CHUNKS) * 8;
             if (key <= last_pos && key >= lo_first) {
-                const T* pg = cache + (size_t)bt[key / page_size] * page_stride;
-                const size_t in_page = (size_t)kvh * page_size + key % page_size;
-                cp_async16(dst, c < CHUNKS ? pg + in_page * HD + c * 8
-                                            : pg + v_base + ((size_t)vh * page_size + key % page_size) * v_stride + (c - CHUNKS) * 8);
+                const int page = page_shift >= 0 ? key >> page_shift : key / page_size, at = key - page * page_size;
+                const T* pg = cache + (size_t)bt[page] * page_stride;
+                cp_async16(dst, c < CHUNKS ? pg + ((size_t)kvh * page_size + at) * HD + c * 8
+                                            : pg + v_base + ((size_t)vh * page_size + at) * v_stride + (c - CHUNKS) * 8);
             } else {                                // never read as a key (masked), but keep the values finite
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
             }
@@ -336,9 +340,11 @@ static int launch_prefill(const void* q, const void* cache, const int32_t* bt, c
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
+    int shift = -1;
+    for (int b = 0; b < 30; b++) if ((1 << b) == page_size) shift = b;
     dim3 grid(n_tiles, nh);
     return launch_plain(kern, grid, dim3(PF_THREADS), smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, tiles,
-                            (__nv_bfloat16*)out, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld);
+                            (__nv_bfloat16*)out, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, shift);
 }
 
 template <int HD>

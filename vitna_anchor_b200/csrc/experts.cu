@@ -79,9 +79,9 @@ __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict_
 
 // A block TB tokens (a row of the router is read once for all of them); a warp a logit, then a warp a token.  all = experts + identities.
 template <typename T, int TB>
-__global__ void __launch_bounds__(128) experts_route_scored_kernel(const T* __restrict__ x, int width, const float* __restrict__ wr,
+__global__ void __launch_bounds__(256) experts_route_scored_kernel(const T* __restrict__ x, int width, const float* __restrict__ wr,
                                                                    const float* __restrict__ correction, int all, int top, int count, int keep, float scale,
-                                                                   int32_t* __restrict__ ids, float* __restrict__ wts, int tokens) {
+                                                                   int32_t* __restrict__ ids, float* __restrict__ wts, int tokens, int vec) {
     extern __shared__ float rs_sm[];                    // [TB][all] scores | [TB][all] choice scores | [TB][count] the groups' best
     dependency_wait();
     let_dependents_start();
@@ -91,10 +91,27 @@ __global__ void __launch_bounds__(128) experts_route_scored_kernel(const T* __re
         float acc[TB];
 #pragma unroll
         for (int b = 0; b < TB; b++) acc[b] = 0.0f;
-        for (int i = lane; i < width; i += 32) {
-            const float wv = w[i];
+        if (vec) {
+            constexpr int V = Vec16<T>::N;
+#pragma unroll 4
+            for (int i = lane * V; i < width; i += 32 * V) {
+                float wv[V];
 #pragma unroll
-            for (int b = 0; b < TB; b++) acc[b] = fmaf(to_f32<T>(x[(size_t)min(t0 + b, tokens - 1) * width + i]), wv, acc[b]);
+                for (int v = 0; v < V; v += 4) *reinterpret_cast<float4*>(wv + v) = *reinterpret_cast<const float4*>(w + i + v);
+#pragma unroll
+                for (int b = 0; b < TB; b++) {
+                    float xv[V];
+                    load16<T>(x + (size_t)min(t0 + b, tokens - 1) * width + i, xv);
+#pragma unroll
+                    for (int v = 0; v < V; v++) acc[b] = fmaf(xv[v], wv[v], acc[b]);
+                }
+            }
+        } else {
+            for (int i = lane; i < width; i += 32) {
+                const float wv = w[i];
+#pragma unroll
+                for (int b = 0; b < TB; b++) acc[b] = fmaf(to_f32<T>(x[(size_t)min(t0 + b, tokens - 1) * width + i]), wv, acc[b]);
+            }
         }
 #pragma unroll
         for (int b = 0; b < TB; b++) {
@@ -179,8 +196,8 @@ __global__ void __launch_bounds__(256) experts_route_table_kernel(const int32_t*
 template <typename T>
 __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restrict__ x, int width, const T* __restrict__ wgu, int ff, int top,
                                                               const int32_t* __restrict__ ids, int E, int act, float limit, float alpha,
-                                                              T* __restrict__ out) {
-    extern __shared__ float xs[];                       // [width]
+                                                              T* __restrict__ out, int vec) {
+    extern __shared__ __align__(16) float xs[];         // [width]
     dependency_wait();
     let_dependents_start();
     const int p = blockIdx.x, t = p / top;
@@ -195,9 +212,25 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
         const T* g = wg + (size_t)c * width;
         const T* u = wu + (size_t)c * width;
         float ag = 0.0f, au = 0.0f;
-        for (int i = lane; i < width; i += 32) {
-            ag = fmaf(xs[i], to_f32<T>(g[i]), ag);
-            au = fmaf(xs[i], to_f32<T>(u[i]), au);
+        if (vec) {                                      // 16 bytes of both rows a lane and step
+            constexpr int V = Vec16<T>::N;
+#pragma unroll 4
+            for (int i = lane * V; i < width; i += 32 * V) {
+                float gv[V], uv[V];
+                load16<T>(g + i, gv);
+                load16<T>(u + i, uv);
+#pragma unroll
+                for (int e = 0; e < V; e += 4) {
+                    const float4 x4 = *reinterpret_cast<const float4*>(xs + i + e);
+                    ag = fmaf(x4.x, gv[e], ag); ag = fmaf(x4.y, gv[e + 1], ag); ag = fmaf(x4.z, gv[e + 2], ag); ag = fmaf(x4.w, gv[e + 3], ag);
+                    au = fmaf(x4.x, uv[e], au); au = fmaf(x4.y, uv[e + 1], au); au = fmaf(x4.z, uv[e + 2], au); au = fmaf(x4.w, uv[e + 3], au);
+                }
+            }
+        } else {
+            for (int i = lane; i < width; i += 32) {
+                ag = fmaf(xs[i], to_f32<T>(g[i]), ag);
+                au = fmaf(xs[i], to_f32<T>(u[i]), au);
+            }
         }
         ag = warp_sum(ag);
         au = warp_sum(au);
@@ -218,8 +251,8 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
 template <typename T>
 __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__ act, int ff, const T* __restrict__ wd, int width, int top,
                                                            const int32_t* __restrict__ ids, const float* __restrict__ wts, float* __restrict__ y, int E,
-                                                           const T* __restrict__ x) {
-    extern __shared__ float as[];                       // [top][ff]
+                                                           const T* __restrict__ x, int vec) {
+    extern __shared__ __align__(16) float as[];         // [top][ff]
     dependency_wait();
     let_dependents_start();
     const int t = blockIdx.x;
@@ -237,7 +270,21 @@ __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__
             const T* w = wd + ((size_t)e * width + c) * ff;
             const float* a = as + (size_t)k * ff;
             float acc = 0.0f;
-            for (int i = lane; i < ff; i += 32) acc = fmaf(a[i], to_f32<T>(w[i]), acc);
+            if (vec) {
+                constexpr int V = Vec16<T>::N;
+#pragma unroll 4
+                for (int i = lane * V; i < ff; i += 32 * V) {
+                    float wv[V];
+                    load16<T>(w + i, wv);
+#pragma unroll
+                    for (int e = 0; e < V; e += 4) {
+                        const float4 a4 = *reinterpret_cast<const float4*>(a + i + e);
+                        acc = fmaf(a4.x, wv[e], acc); acc = fmaf(a4.y, wv[e + 1], acc); acc = fmaf(a4.z, wv[e + 2], acc); acc = fmaf(a4.w, wv[e + 3], acc);
+                    }
+                }
+            } else {
+                for (int i = lane; i < ff; i += 32) acc = fmaf(a[i], to_f32<T>(w[i]), acc);
+            }
             total = fmaf(wts[(size_t)t * top + k], warp_sum(acc), total);
         }
         if (lane == 0) y[(size_t)t * width + c] += total;
@@ -310,6 +357,29 @@ __global__ void __launch_bounds__(256) experts_combine_kernel(const float* __res
     dependency_wait();
     let_dependents_start();
     const int t = blockIdx.x;
+    if (width % 4 == 0 && ((uintptr_t)o % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)x % 16) == 0) {
+        for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
+            float4 sum = *reinterpret_cast<const float4*>(y + (size_t)t * width + c);
+            float4 total = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            for (int k = 0; k < top; k++) {
+                const int r = pos[(size_t)t * top + k];
+                const float w = wts[(size_t)t * top + k];
+                float4 v;
+                if (r >= 0) {
+                    v = *reinterpret_cast<const float4*>(o + (size_t)r * width + c);
+                } else if (ids[(size_t)t * top + k] >= E) {
+                    const T* p = x + (size_t)t * width + c;
+                    v = make_float4(to_f32<T>(p[0]), to_f32<T>(p[1]), to_f32<T>(p[2]), to_f32<T>(p[3]));
+                } else {
+                    continue;
+                }
+                total.x = fmaf(w, v.x, total.x); total.y = fmaf(w, v.y, total.y); total.z = fmaf(w, v.z, total.z); total.w = fmaf(w, v.w, total.w);
+            }
+            sum.x += total.x; sum.y += total.y; sum.z += total.z; sum.w += total.w;
+            *reinterpret_cast<float4*>(y + (size_t)t * width + c) = sum;
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float total = 0.0f;
         for (int k = 0; k < top; k++) {
@@ -372,9 +442,10 @@ VK_API int vk_experts_route_scored(const void* x, int width, const float* wr, co
     const size_t smem = (size_t)tb * (2 * all + count) * sizeof(float);
     if (smem > 48 * 1024) return VK_TOO_LARGE;
     const dim3 grid((tokens + tb - 1) / tb);
+    const int vec = width % (dtype == 0 ? 4 : 8) == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)wr % 16) == 0;
 #define VK_ERS(T, TB)                                                                                                                          \
-    return launch_dependent(experts_route_scored_kernel<T, TB>, grid, dim3(128), smem, stream, (const T*)x, width, wr, correction, all, top, count, \
-                            keep, scale, ids, wts, tokens)
+    return launch_dependent(experts_route_scored_kernel<T, TB>, grid, dim3(256), smem, stream, (const T*)x, width, wr, correction, all, top, count, \
+                            keep, scale, ids, wts, tokens, vec)
     if (dtype == 0) {
         if (tb == 4) VK_ERS(float, 4);
         VK_ERS(float, 1);
@@ -416,11 +487,12 @@ VK_API int vk_experts_gate_up(const void* x, int width, const void* wgu, int ff,
     int gy = (ff + 7) / 8;
     if (gy > 64) gy = 64;
     dim3 grid(tokens * top, gy);
+    const int vec = width % (dtype == 0 ? 4 : 8) == 0 && ((uintptr_t)wgu % 16) == 0;
     if (dtype == 0)
         return launch_dependent(experts_gate_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, width, (const float*)wgu, ff, top, ids, E, act,
-                                limit, alpha, (float*)out);
+                                limit, alpha, (float*)out, vec);
     return launch_dependent(experts_gate_up_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, width,
-                            (const __nv_bfloat16*)wgu, ff, top, ids, E, act, limit, alpha, (__nv_bfloat16*)out);
+                            (const __nv_bfloat16*)wgu, ff, top, ids, E, act, limit, alpha, (__nv_bfloat16*)out, vec);
 }
 
 // act [tokens * top][ff] and wd [E][width][ff] in dtype; y float32 [tokens][width] is added to; ids of E and more: the token's row of x.
@@ -433,6 +505,7 @@ VK_API int vk_experts_down(const void* act, int ff, const void* wd, int width, i
     int gy = (width + 7) / 8;
     if (gy > 64) gy = 64;
     dim3 grid(tokens, gy);
+    const int vec = ff % (dtype == 0 ? 4 : 8) == 0 && ((uintptr_t)wd % 16) == 0;
     if (smem > 48 * 1024) {
         cudaError_t e = dtype == 0 ? cudaFuncSetAttribute(experts_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
                                    : cudaFuncSetAttribute(experts_down_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -440,7 +513,7 @@ VK_API int vk_experts_down(const void* act, int ff, const void* wd, int width, i
     }
     if (dtype == 0)
         return launch_dependent(experts_down_kernel<float>, grid, dim3(256), smem, stream, (const float*)act, ff, (const float*)wd, width, top, ids, wts, y,
-                                E, (const float*)x);
+                                E, (const float*)x, vec);
     return launch_dependent(experts_down_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)act, ff, (const __nv_bfloat16*)wd,
-                            width, top, ids, wts, y, E, (const __nv_bfloat16*)x);
+                            width, top, ids, wts, y, E, (const __nv_bfloat16*)x, vec);
 }

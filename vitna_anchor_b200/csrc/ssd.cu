@@ -261,20 +261,36 @@ __global__ void __launch_bounds__(256) ssd_decode_kernel(const float* __restrict
     }
 }
 
+template <typename T> __device__ __forceinline__ void ssd_store4(T* p, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void ssd_store4<float>(float* p, float a, float b, float c, float d) {
+    *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+template <> __device__ __forceinline__ void ssd_store4<__nv_bfloat16>(__nv_bfloat16* p, float a, float b, float c, float d) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) ssd_gate_kernel(const float* __restrict__ y, const float* __restrict__ proj, int N, int z_off, int x_off,
                                                        const float* __restrict__ w, float eps, float mult, int inner, int parts, T* __restrict__ out,
                                                        int out_ld, const int32_t* __restrict__ token_seg, const int32_t* __restrict__ seg_starts,
                                                        const int32_t* __restrict__ seg_slots, float* __restrict__ state, size_t state_stride,
-                                                       size_t conv_off, int C, int taps) {
-    extern __shared__ float sg_sm[];                        // [inner] gated values, [parts] 1 / rms
+                                                       size_t conv_off, int C, int taps, int vec) {
+    extern __shared__ __align__(16) float sg_sm[];          // [inner] gated values, [parts] 1 / rms
     __shared__ float scratch[32];
     float* inv = sg_sm + inner;
     dependency_wait();
     let_dependents_start();
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const float* in = proj + (size_t)t * N;
-    for (int i = tid; i < inner; i += 256) sg_sm[i] = y[(size_t)t * inner + i] * silu_f(in[z_off + i]);
+    if (vec) {
+        for (int i = tid * 4; i < inner; i += 1024) {
+            const float4 a = *reinterpret_cast<const float4*>(y + (size_t)t * inner + i), z = *reinterpret_cast<const float4*>(in + z_off + i);
+            *reinterpret_cast<float4*>(sg_sm + i) = make_float4(a.x * silu_f(z.x), a.y * silu_f(z.y), a.z * silu_f(z.z), a.w * silu_f(z.w));
+        }
+    } else {
+        for (int i = tid; i < inner; i += 256) sg_sm[i] = y[(size_t)t * inner + i] * silu_f(in[z_off + i]);
+    }
     const int size = inner / parts;
     __syncthreads();
     if (parts >= 8) {
@@ -294,7 +310,15 @@ __global__ void __launch_bounds__(256) ssd_gate_kernel(const float* __restrict__
     }
     __syncthreads();
     T* dst = out + (size_t)t * out_ld;
-    for (int i = tid; i < inner; i += 256) dst[i] = from_f32<T>((sg_sm[i] * inv[i / size]) * w[i]);
+    if (vec && size % 4 == 0) {
+        for (int i = tid * 4; i < inner; i += 1024) {
+            const float4 a = *reinterpret_cast<const float4*>(sg_sm + i), ww = *reinterpret_cast<const float4*>(w + i);
+            const float r = inv[i / size];
+            ssd_store4<T>(dst + i, (a.x * r) * ww.x, (a.y * r) * ww.y, (a.z * r) * ww.z, (a.w * r) * ww.w);
+        }
+    } else {
+        for (int i = tid; i < inner; i += 256) dst[i] = from_f32<T>((sg_sm[i] * inv[i / size]) * w[i]);
+    }
     // the convolution's memory: the last taps - 1 inputs, of which a short step may leave some of the old ones
     const int seg = token_seg[t], first = seg_starts[seg], end = seg_starts[seg + 1], slot = seg_slots[seg];
     if (t != end - 1 || slot < 0 || taps < 2) return;
@@ -422,6 +446,8 @@ VK_API int vk_ssd_gate(const float* y, const float* proj, int N_proj, int z_off,
     if (smem > 200 * 1024) return VK_TOO_LARGE;
     const bool few = tokens <= DR_DEPENDENT_TOKENS;
     const size_t conv_off = (size_t)H * N * P;
+    const int vec = inner % 4 == 0 && N_proj % 4 == 0 && z_off % 4 == 0 && out_ld % 4 == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)proj % 16) == 0 &&
+                    ((uintptr_t)w % 16) == 0 && ((uintptr_t)out % (dtype == 0 ? 16 : 8)) == 0;
 #define VK_SSDG(T)                                                                                                                           \
     do {                                                                                                                                     \
         auto kern = ssd_gate_kernel<T>;                                                                                                      \
@@ -430,7 +456,7 @@ VK_API int vk_ssd_gate(const float* y, const float* proj, int N_proj, int z_off,
             if (e != cudaSuccess) return (int)e;                                                                                             \
         }                                                                                                                                    \
         return ssd_launch(few, kern, dim3(tokens), dim3(256), smem, stream, y, proj, N_proj, z_off, x_off, w, eps, mult, inner, parts, (T*)out, \
-                          out_ld, token_seg, seg_starts, seg_slots, state, state_stride, conv_off, C, taps);                                 \
+                          out_ld, token_seg, seg_starts, seg_slots, state, state_stride, conv_off, C, taps, vec);                            \
     } while (0)
     if (dtype == 0) VK_SSDG(float);
     VK_SSDG(__nv_bfloat16);

@@ -258,6 +258,23 @@ __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ 
     dependency_wait();
     let_dependents_start();
     const T* row = gu + (size_t)blockIdx.x * 2 * inter;
+    constexpr int V = Vec16<T>::N;
+    if (inter % V == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)out % 16) == 0) {
+        for (int i = threadIdx.x * V; i < inter; i += blockDim.x * V) {
+            float g[V], u[V];
+            load16<T>(row + i, g);
+            load16<T>(row + inter + i, u);
+#pragma unroll
+            for (int e = 0; e < V; e++) {
+                const float gg = fminf(g[e], limit), uu = fminf(fmaxf(u[e], -limit), limit);
+                g[e] = (gg / (1.0f + expf(-alpha * gg))) * (uu + 1.0f);
+            }
+            T* dst = out + (size_t)blockIdx.x * inter + i;
+#pragma unroll
+            for (int e = 0; e < V; e += 4) sw_store4<T>(dst + e, g[e], g[e + 1], g[e + 2], g[e + 3]);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < inter; i += blockDim.x) {
         const float g = fminf(to_f32<T>(row[i]), limit);
         const float u = fminf(fmaxf(to_f32<T>(row[inter + i]), -limit), limit);
