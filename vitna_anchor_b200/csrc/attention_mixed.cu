@@ -92,6 +92,98 @@ __global__ void __launch_bounds__(256) mixed_attn_prepare_kernel(const float* __
     }
 }
 
+template <typename T> __device__ __forceinline__ void am_store4(T* p, float4 v);
+template <> __device__ __forceinline__ void am_store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void am_store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+template <typename T> __device__ __forceinline__ void am_store2(T* p, float a, float b);
+template <> __device__ __forceinline__ void am_store2<float>(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+template <> __device__ __forceinline__ void am_store2<__nv_bfloat16>(__nv_bfloat16* p, float a, float b) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
+// mixed_attn_prepare without norms and with unturned values, where every size is a multiple of four and everything lies on 16 bytes: a thread
+// takes four values at a time (two pairs of a turned part, or four neighbours), whose inputs are asked for before the angles are worked out.
+template <typename T>
+__global__ void __launch_bounds__(256) rotary_store_kernel(const float* __restrict__ proj, int N, const int32_t* __restrict__ positions,
+                                                           const int32_t* __restrict__ slot, const float* __restrict__ freq, int dims,
+                                                           T* __restrict__ q_out, T* __restrict__ cache, int nh, int nkv, int hd, int vd, int page_size,
+                                                           const float* __restrict__ bias, float v_mult) {
+    extern __shared__ float rs_turn[];                  // [dims/2][2] cos and sin of the token's angles
+    constexpr int U = 3;                                // items of a thread on their way together
+    dependency_wait();
+    let_dependents_start();
+    const int t = blockIdx.x, tid = threadIdx.x, half = dims / 2;
+    const float* in = proj + (size_t)t * N;
+    const int per_head = hd / 4, turned = dims / 4, n_qk = (nh + nkv) * per_head, total = n_qk + nkv * vd / 4;
+    // item i -> columns (a pair of float2, or one float4)
+    auto fetch = [&](int i, float4& v) {
+        if (i >= n_qk) {
+            const int c = (nh + nkv) * hd + (i - n_qk) * 4;
+            v = *reinterpret_cast<const float4*>(in + c);
+            if (bias) { const float4 b = *reinterpret_cast<const float4*>(bias + c); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+            return;
+        }
+        const int h = i / per_head, j = i - h * per_head;
+        if (j < turned) {
+            const int c = h * hd + 2 * j;
+            const float2 a = *reinterpret_cast<const float2*>(in + c), b = *reinterpret_cast<const float2*>(in + c + half);
+            v = make_float4(a.x, a.y, b.x, b.y);
+            if (bias) {
+                const float2 ba = *reinterpret_cast<const float2*>(bias + c), bb = *reinterpret_cast<const float2*>(bias + c + half);
+                v.x += ba.x; v.y += ba.y; v.z += bb.x; v.w += bb.y;
+            }
+        } else {
+            const int c = h * hd + 4 * j;
+            v = *reinterpret_cast<const float4*>(in + c);
+            if (bias) { const float4 b = *reinterpret_cast<const float4*>(bias + c); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+        }
+    };
+    const int s = (slot && cache) ? slot[t] : -1;
+    const size_t page_stride = (size_t)nkv * page_size * (hd + vd);
+    T* kbase = s >= 0 ? cache + (size_t)(s / page_size) * page_stride : nullptr;
+    T* vbase = s >= 0 ? kbase + (size_t)nkv * page_size * hd : nullptr;
+    const int off = s >= 0 ? s % page_size : 0;
+    float4 v[U];
+#pragma unroll
+    for (int u = 0; u < U; u++)
+        if (tid + u * 256 < total) fetch(tid + u * 256, v[u]);
+    const float pos = (float)positions[t];
+    for (int i = tid; i < half; i += 256) {
+        const float ang = pos * freq[i];
+        rs_turn[2 * i] = cosf(ang);
+        rs_turn[2 * i + 1] = sinf(ang);
+    }
+    __syncthreads();
+    for (int base = tid; base < total; base += U * 256) {
+#pragma unroll
+        for (int u = 0; u < U; u++) {
+            const int i = base + u * 256;
+            if (i >= total) break;
+            if (base != tid) fetch(i, v[u]);
+            if (i >= n_qk) {
+                if (s >= 0) {
+                    const int e = (i - n_qk) * 4, g = e / vd, d = e - g * vd;
+                    am_store4<T>(vbase + ((size_t)g * page_size + off) * vd + d, make_float4(v[u].x * v_mult, v[u].y * v_mult, v[u].z * v_mult, v[u].w * v_mult));
+                }
+                continue;
+            }
+            const int h = i / per_head, j = i - h * per_head;
+            T* dst = h < nh ? q_out + ((size_t)t * nh + h) * hd : (s >= 0 ? kbase + ((size_t)(h - nh) * page_size + off) * hd : nullptr);
+            if (!dst) continue;
+            if (j < turned) {
+                const float c0 = rs_turn[4 * j], s0 = rs_turn[4 * j + 1], c1 = rs_turn[4 * j + 2], s1 = rs_turn[4 * j + 3];
+                am_store2<T>(dst + 2 * j, v[u].x * c0 - v[u].z * s0, v[u].y * c1 - v[u].w * s1);
+                am_store2<T>(dst + 2 * j + half, v[u].z * c0 + v[u].x * s0, v[u].w * c1 + v[u].y * s1);
+            } else {
+                am_store4<T>(dst + 4 * j, v[u]);
+            }
+        }
+    }
+}
+
 // PARTIAL: the block takes the runs  blockIdx.y * runs_per_split ..  of its token's keys alone and leaves, instead of the output,
 // the unnormalised sums, the maximum and the sum of the weights of every head in part [token][split][nh * (vd + 2)]
 // (attention_mixed_combine adds the splits up): single decoded tokens far into a context are spread over many blocks.
@@ -619,6 +711,15 @@ VK_API int vk_mixed_attn_prepare(const float* proj, int N, const int32_t* positi
         return VK_BAD_SHAPE;
     const size_t smem = (size_t)(dims + vd + 1) * sizeof(float);
     if (smem > 48 * 1024) return VK_TOO_LARGE;
+    auto on16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+    if (eps < 0.0f && !qn_w && !kn_w && !vfreq && hd % 4 == 0 && vd % 4 == 0 && dims % 4 == 0 && N % 4 == 0 && on16(proj) && on16(q_out) && on16(cache) &&
+        on16(bias)) {
+        if (dtype == 0)
+            return launch_dependent(rotary_store_kernel<float>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, freq, dims, (float*)q_out,
+                                    (float*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);
+        return launch_dependent(rotary_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, freq, dims,
+                                (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);
+    }
     if (dtype == 0)
         return launch_dependent(mixed_attn_prepare_kernel<float>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
                                 dims, vfreq, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);

@@ -14,8 +14,8 @@
 //                  form of the exact 32-bit routing and of the sizes that the chunked form (ssd_chunked.cu) does not take.
 //  ssd_decode      single tokens: convolution, gates, one step and the state's update in one launch, a block per (columns, head,
 //                  segment); the state's rows are on their way before the kernel waits for the product in front of it.
-//  ssd_gate        a block a token: gate, norm, weight, to columns of the output product's input; the block of a segment's last token
-//                  moves the convolution's memory on (nothing after it in the step reads the old one).
+//  ssd_gate        a block a token: gate, norm, weight, to columns of the output product's input; further blocks move the convolution's
+//                  memory of the segments on (nothing after them in the step reads the old one).
 //
 // A request's state row: S float32 [H][N][P], then the last taps - 1 inputs of the convolution, float32 [taps - 1][H P + 2 G N].
 // Everything is float32 with accurate expf and log1pf; only what the convolution gives is rounded to the compute dtype.
@@ -54,6 +54,9 @@ __global__ void __launch_bounds__(256) ssd_prepare_kernel(const float* __restric
     for (int i = 0; i < SSD_PREP_TOKENS; i++) in[i] = i < cnt ? proj[(size_t)(t0 + i) * N + x_off + c] : 0.0f;
 #pragma unroll
     for (int j = 0; j < MT; j++) w[j] = j < taps ? conv_w[(size_t)c * taps + (taps - 1 - j)] : 0.0f;
+    float before[MT - 1];                                   // the rows in front of the block's first token, if they are the same request's
+#pragma unroll
+    for (int j = 0; j < MT - 1; j++) before[j] = (j < taps - 1 && t0 - (j + 1) >= 0) ? proj[(size_t)(t0 - (j + 1)) * N + x_off + c] : 0.0f;
     const float b = conv_b ? conv_b[c] : 0.0f;
     int seg = -1;
 #pragma unroll
@@ -69,7 +72,7 @@ __global__ void __launch_bounds__(256) ssd_prepare_kernel(const float* __restric
                     x[j] = 0.0f;
                     if (j < taps - 1) {
                         const int src = at - (j + 1);
-                        if (src >= 0) x[j] = proj[(size_t)(t - (j + 1)) * N + x_off + c];
+                        if (src >= 0) x[j] = before[j];     // only at the block's first token: any other that begins here is its request's first
                         else if (old) x[j] = old[(size_t)(taps - 1 + src) * C + c];
                     }
                 }
@@ -273,14 +276,30 @@ template <> __device__ __forceinline__ void ssd_store4<__nv_bfloat16>(__nv_bfloa
 template <typename T>
 __global__ void __launch_bounds__(256) ssd_gate_kernel(const float* __restrict__ y, const float* __restrict__ proj, int N, int z_off, int x_off,
                                                        const float* __restrict__ w, float eps, float mult, int inner, int parts, T* __restrict__ out,
-                                                       int out_ld, const int32_t* __restrict__ token_seg, const int32_t* __restrict__ seg_starts,
-                                                       const int32_t* __restrict__ seg_slots, float* __restrict__ state, size_t state_stride,
-                                                       size_t conv_off, int C, int taps, int vec) {
+                                                       int out_ld, const int32_t* __restrict__ seg_starts, const int32_t* __restrict__ seg_slots,
+                                                       float* __restrict__ state, size_t state_stride, size_t conv_off, int C, int taps, int vec, int tokens) {
     extern __shared__ __align__(16) float sg_sm[];          // [inner] gated values, [parts] 1 / rms
     __shared__ float scratch[32];
     float* inv = sg_sm + inner;
     dependency_wait();
     let_dependents_start();
+    if (blockIdx.x >= tokens) {                             // the convolution's memory: a thread a channel of a segment
+        const int per = (C + 255) / 256, seg = (blockIdx.x - tokens) / per, c = (blockIdx.x - tokens) % per * 256 + threadIdx.x;
+        const int first = seg_starts[seg], n = seg_starts[seg + 1] - first, slot = seg_slots[seg];
+        if (slot < 0 || n <= 0 || c >= C) return;
+        float* mem = state + (size_t)slot * state_stride + conv_off + c;
+        float v[DR_MAX_TAPS];                               // the last taps - 1 inputs, of which a short step leaves some of the old ones
+#pragma unroll
+        for (int j = 0; j < DR_MAX_TAPS; j++)
+            if (j < taps - 1) {
+                const int src = n - (taps - 1) + j;
+                v[j] = src >= 0 ? proj[(size_t)(first + src) * N + x_off + c] : mem[(size_t)(j + n) * C];
+            }
+#pragma unroll
+        for (int j = 0; j < DR_MAX_TAPS; j++)
+            if (j < taps - 1) mem[(size_t)j * C] = v[j];
+        return;
+    }
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const float* in = proj + (size_t)t * N;
     if (vec) {
@@ -319,16 +338,6 @@ __global__ void __launch_bounds__(256) ssd_gate_kernel(const float* __restrict__
     } else {
         for (int i = tid; i < inner; i += 256) dst[i] = from_f32<T>((sg_sm[i] * inv[i / size]) * w[i]);
     }
-    // the convolution's memory: the last taps - 1 inputs, of which a short step may leave some of the old ones
-    const int seg = token_seg[t], first = seg_starts[seg], end = seg_starts[seg + 1], slot = seg_slots[seg];
-    if (t != end - 1 || slot < 0 || taps < 2) return;
-    const int n = end - first;
-    float* mem = state + (size_t)slot * state_stride + conv_off;
-    for (int c = tid; c < C; c += 256)
-        for (int j = 0; j < taps - 1; j++) {
-            const int src = n - (taps - 1) + j;             // place in this step's portion; before it: an input of an earlier step
-            mem[(size_t)j * C + c] = src >= 0 ? proj[(size_t)(first + src) * N + x_off + c] : mem[(size_t)(j + n) * C + c];
-        }
 }
 
 template <typename... KArgs, typename... Args>
@@ -435,8 +444,7 @@ VK_API int vk_ssd_decode(const float* proj, int N_proj, int x_off, int dt_off, c
 // out (rows out_ld apart, H P columns each) in dtype = mult * rms-normed (in `parts` equal parts) (y silu(z)) * w; moves the convolution's
 // memory of every segment on.
 VK_API int vk_ssd_gate(const float* y, const float* proj, int N_proj, int z_off, int x_off, const float* w, float eps, float mult, int parts, void* out,
-                       int out_ld, const int32_t* token_seg, const int32_t* seg_starts, const int32_t* seg_slots, float* state, size_t state_stride,
-                       int tokens, int H, int G, int N, int P, int taps, int dtype, cudaStream_t stream) {
+                       int out_ld, const int32_t* seg_starts, const int32_t* seg_slots, int segments, float* state, size_t state_stride, int tokens, int H, int G, int N, int P, int taps, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     const int C = H * P + 2 * G * N, inner = H * P;
     if (!ssd_sizes_ok(H, G, N, P, taps) || parts <= 0 || inner % parts || z_off < 0 || z_off + inner > N_proj || x_off < 0 || x_off + C > N_proj ||
@@ -448,6 +456,7 @@ VK_API int vk_ssd_gate(const float* y, const float* proj, int N_proj, int z_off,
     const size_t conv_off = (size_t)H * N * P;
     const int vec = inner % 4 == 0 && N_proj % 4 == 0 && z_off % 4 == 0 && out_ld % 4 == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)proj % 16) == 0 &&
                     ((uintptr_t)w % 16) == 0 && ((uintptr_t)out % (dtype == 0 ? 16 : 8)) == 0;
+    const dim3 grid(tokens + (taps > 1 ? segments * ((C + 255) / 256) : 0));
 #define VK_SSDG(T)                                                                                                                           \
     do {                                                                                                                                     \
         auto kern = ssd_gate_kernel<T>;                                                                                                      \
@@ -455,8 +464,8 @@ VK_API int vk_ssd_gate(const float* y, const float* proj, int N_proj, int z_off,
             cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                              \
             if (e != cudaSuccess) return (int)e;                                                                                             \
         }                                                                                                                                    \
-        return ssd_launch(few, kern, dim3(tokens), dim3(256), smem, stream, y, proj, N_proj, z_off, x_off, w, eps, mult, inner, parts, (T*)out, \
-                          out_ld, token_seg, seg_starts, seg_slots, state, state_stride, conv_off, C, taps, vec);                            \
+        return ssd_launch(few, kern, grid, dim3(256), smem, stream, y, proj, N_proj, z_off, x_off, w, eps, mult, inner, parts, (T*)out, \
+                          out_ld, seg_starts, seg_slots, state, state_stride, conv_off, C, taps, vec, tokens);                               \
     } while (0)
     if (dtype == 0) VK_SSDG(float);
     VK_SSDG(__nv_bfloat16);

@@ -80,14 +80,15 @@ __device__ __forceinline__ SscChunk ssc_find(int n, const int32_t* __restrict__ 
     return SscChunk{sh[0], sh[1], sh[2]};
 }
 
-// rows x cols bfloat16 from src (rows ld apart) into dst (rows dst_ld apart), zeros up to rows_pad x cols_pad (cols_pad a multiple of 8)
-__device__ __forceinline__ void ssc_tile(__nv_bfloat16* dst, int dst_ld, const __nv_bfloat16* __restrict__ src, size_t ld, int rows, int cols, int rows_pad,
-                                         int cols_pad) {
+// rows x cols bfloat16 from src (rows ld apart) into dst (rows COLS + 8 apart), zeros up to ROWS x COLS (COLS a multiple of 8)
+template <int ROWS, int COLS>
+__device__ __forceinline__ void ssc_tile(__nv_bfloat16* dst, const __nv_bfloat16* __restrict__ src, size_t ld, int rows, int cols) {
     const bool vec = (reinterpret_cast<uintptr_t>(src) % 16 == 0) && ld % 8 == 0 && cols % 8 == 0;
-    const int pieces = cols_pad / 8;
-    for (int i = threadIdx.x; i < rows_pad * pieces; i += SC_THREADS) {
-        const int r = i / pieces, c = (i % pieces) * 8;
-        __nv_bfloat16* d = dst + r * dst_ld + c;
+    constexpr int PIECES = COLS / 8;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < ROWS * PIECES; i += SC_THREADS) {
+        const int r = i / PIECES, c = (i % PIECES) * 8;
+        __nv_bfloat16* d = dst + r * (COLS + 8) + c;
         if (r < rows && c < cols && vec) {
             dr_cp_async16(d, src + r * ld + c);
         } else {
@@ -126,13 +127,15 @@ __device__ __forceinline__ void ssc_gates(float* L, float* dt, const float* __re
     }
 }
 
+// NP: the state's rows, rounded up to a size that is built
+template <int NP>
 __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_state_kernel(const __nv_bfloat16* __restrict__ xbc, const float* __restrict__ gates,
                                                                      const int32_t* __restrict__ seg_starts, int segments, float* __restrict__ add,
                                                                      float* __restrict__ whole, int C, int H, int G, int N, int P) {
     extern __shared__ __align__(16) unsigned char ss_raw[];
     __shared__ float L[SC_Q], dt[SC_Q];
     __shared__ int find[3];
-    const int NP = (N + 15) / 16 * 16, LDB = NP + 8;
+    constexpr int LDB = NP + 8;
     __nv_bfloat16* sb = reinterpret_cast<__nv_bfloat16*>(ss_raw);       // [64][LDB]
     __nv_bfloat16* sx = sb + SC_Q * LDB;                                // [64][SC_LD] high parts of w x (first: x itself)
     __nv_bfloat16* sl = sx + SC_Q * SC_LD;                              // [64][SC_LD] low parts
@@ -140,8 +143,8 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_state_kernel(const __nv_
     if (ch.seg < 0) return;
     const int h = blockIdx.y, p0 = blockIdx.z * SC_P, pc = min(SC_P, P - p0), g = h / (H / G);
     const __nv_bfloat16* base = xbc + (size_t)ch.first * C;
-    ssc_tile(sb, LDB, base + H * P + g * N, C, ch.rows, N, SC_Q, NP);
-    ssc_tile(sx, SC_LD, base + h * P + p0, C, ch.rows, pc, SC_Q, SC_P);
+    ssc_tile<SC_Q, NP>(sb, base + H * P + g * N, C, ch.rows, N);
+    ssc_tile<SC_Q, SC_P>(sx, base + h * P + p0, C, ch.rows, pc);
     asm volatile("cp.async.commit_group;" ::: "memory");
     ssc_gates(L, dt, gates, ch.first, ch.rows, H, h);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -260,6 +263,7 @@ __global__ void __launch_bounds__(256) ssd_chunk_scan_kernel(const float* __rest
     else *st = s[0];
 }
 
+template <int NP>
 __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(const __nv_bfloat16* __restrict__ xbc, const float* __restrict__ gates,
                                                                    const float* __restrict__ D, const int32_t* __restrict__ seg_starts, int segments,
                                                                    const __nv_bfloat16* __restrict__ hi, const __nv_bfloat16* __restrict__ lo,
@@ -267,7 +271,7 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(const __nv_bf
     extern __shared__ __align__(16) unsigned char so_raw[];
     __shared__ float L[SC_Q], dt[SC_Q];
     __shared__ int find[3];
-    const int NP = (N + 15) / 16 * 16, LDB = NP + 8;
+    constexpr int LDB = NP + 8;
     __nv_bfloat16* sc = reinterpret_cast<__nv_bfloat16*>(so_raw);       // [64][LDB]
     __nv_bfloat16* sb = sc + SC_Q * LDB;                                // [64][LDB]
     __nv_bfloat16* sx = sb + SC_Q * LDB;                                // [64][SC_LD]
@@ -278,11 +282,11 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(const __nv_bf
     const int h = blockIdx.y, p0 = blockIdx.z * SC_P, pc = min(SC_P, P - p0), g = h / (H / G);
     const __nv_bfloat16* base = xbc + (size_t)ch.first * C;
     const size_t st = ((size_t)blockIdx.x * H + h) * N * P + p0;
-    ssc_tile(sc, LDB, base + H * P + G * N + g * N, C, ch.rows, N, SC_Q, NP);
-    ssc_tile(sb, LDB, base + H * P + g * N, C, ch.rows, N, SC_Q, NP);
-    ssc_tile(sx, SC_LD, base + h * P + p0, C, ch.rows, pc, SC_Q, SC_P);
-    ssc_tile(sh, SC_LD, hi + st, P, N, pc, NP, SC_P);
-    ssc_tile(sl, SC_LD, lo + st, P, N, pc, NP, SC_P);
+    ssc_tile<SC_Q, NP>(sc, base + H * P + G * N + g * N, C, ch.rows, N);
+    ssc_tile<SC_Q, NP>(sb, base + H * P + g * N, C, ch.rows, N);
+    ssc_tile<SC_Q, SC_P>(sx, base + h * P + p0, C, ch.rows, pc);
+    ssc_tile<NP, SC_P>(sh, hi + st, P, N, pc);
+    ssc_tile<NP, SC_P>(sl, lo + st, P, N, pc);
     asm volatile("cp.async.commit_group;" ::: "memory");
     ssc_gates(L, dt, gates, ch.first, ch.rows, H, h);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -295,6 +299,7 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(const __nv_bf
         s[nb][0] = s[nb][1] = s[nb][2] = s[nb][3] = 0.0f;
         o[nb][0] = o[nb][1] = o[nb][2] = o[nb][3] = 0.0f;
     }
+#pragma unroll
     for (int kt = 0; kt < NP / 16; kt++) {
         uint32_t a[4];
         sc_ldsm4(a, sc + (warp * 16 + (lane & 15)) * LDB + kt * 16 + (lane >> 4) * 8);
@@ -373,14 +378,9 @@ using namespace vk;
 
 static int ssc_chunks(int tokens, int segments) { return tokens / SC_Q + (segments < tokens ? segments : tokens); }
 static size_t ssc_up(size_t b) { return (b + 255) / 256 * 256; }
-static size_t ssc_state_smem(int N) {
-    const int NP = (N + 15) / 16 * 16;
-    return (size_t)(SC_Q * (NP + 8) + 2 * SC_Q * SC_LD) * 2;
-}
-static size_t ssc_out_smem(int N) {
-    const int NP = (N + 15) / 16 * 16;
-    return (size_t)(2 * SC_Q * (NP + 8) + SC_Q * SC_LD + 2 * NP * SC_LD) * 2;
-}
+static int ssc_rows(int N) { return N <= 16 ? 16 : N <= 32 ? 32 : N <= 64 ? 64 : N <= 128 ? 128 : 256; }     // the sizes that are built
+static size_t ssc_state_smem(int NP) { return (size_t)(SC_Q * (NP + 8) + 2 * SC_Q * SC_LD) * 2; }
+static size_t ssc_out_smem(int NP) { return (size_t)(2 * SC_Q * (NP + 8) + SC_Q * SC_LD + 2 * NP * SC_LD) * 2; }
 
 VK_API size_t vk_ssd_chunked_scratch_bytes(int tokens, int segments, int H, int N, int P) {
     const size_t chunks = ssc_chunks(tokens, segments), states = chunks * H * N * P;
@@ -401,12 +401,16 @@ VK_API int vk_ssd_chunked(const void* xbc, const float* gates, const float* D, c
     __nv_bfloat16* lo = (__nv_bfloat16*)((char*)hi + ssc_up(states * 2));
     float* whole = (float*)((char*)lo + ssc_up(states * 2));
     dim3 grid(chunks, H, (P + SC_P - 1) / SC_P);
-    const size_t smem1 = ssc_state_smem(N), smem3 = ssc_out_smem(N);
-    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(ssd_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+    const int NP = ssc_rows(N);
+    const size_t smem1 = ssc_state_smem(NP), smem3 = ssc_out_smem(NP);
+    auto state_kernel = NP == 16 ? ssd_chunk_state_kernel<16> : NP == 32 ? ssd_chunk_state_kernel<32> : NP == 64 ? ssd_chunk_state_kernel<64>
+                      : NP == 128 ? ssd_chunk_state_kernel<128> : ssd_chunk_state_kernel<256>;
+    auto out_kernel = NP == 16 ? ssd_chunk_out_kernel<16> : NP == 32 ? ssd_chunk_out_kernel<32> : NP == 64 ? ssd_chunk_out_kernel<64>
+                    : NP == 128 ? ssd_chunk_out_kernel<128> : ssd_chunk_out_kernel<256>;
+    cudaError_t e = cudaFuncSetAttribute(state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
     if (e != cudaSuccess) return (int)e;
-    int s = launch_plain(ssd_chunk_state_kernel, grid, dim3(SC_THREADS), smem1, stream, (const __nv_bfloat16*)xbc, gates, seg_starts, segments, add, whole,
-                         C, H, G, N, P);
+    int s = launch_plain(state_kernel, grid, dim3(SC_THREADS), smem1, stream, (const __nv_bfloat16*)xbc, gates, seg_starts, segments, add, whole, C, H, G, N, P);
     if (s != VK_OK) return s;
     const int NPe = N * P;
     if (NPe % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state % 16) == 0)
@@ -416,6 +420,6 @@ VK_API int vk_ssd_chunked(const void* xbc, const float* gates, const float* D, c
         s = launch_plain(ssd_chunk_scan_kernel<1>, dim3((NPe + 255) / 256, H, segments), dim3(256), 0, stream, add, whole, seg_starts, seg_slots, state,
                          state_stride, hi, lo, H, NPe);
     if (s != VK_OK) return s;
-    return launch_plain(ssd_chunk_out_kernel, grid, dim3(SC_THREADS), smem3, stream, (const __nv_bfloat16*)xbc, gates, D, seg_starts, segments, hi, lo, y, C,
+    return launch_plain(out_kernel, grid, dim3(SC_THREADS), smem3, stream, (const __nv_bfloat16*)xbc, gates, D, seg_starts, segments, hi, lo, y, C,
                         H, G, N, P);
 }

@@ -1822,5 +1822,5 @@ def ssd(proj: torch.Tensor, off: int, conv_w: torch.Tensor, conv_b: Optional[tor
             _check(L.vk_ssd_recurrence(_p(xbc), _p(gates), _p(D), _p(ctx.seg_starts), _p(ctx.seg_slots), _p(state), stride, _p(y), ctx.num_segments, H, G,
                                        N, P, _dt(out), _stream()), "ssd_recurrence")
     _check(L.vk_ssd_gate(_p(y), _p(proj), width, z_off, x_off, _p(norm_w), ctypes.c_float(eps), ctypes.c_float(mult), parts, _p(out), out_ld,
-                         _p(ctx.token_seg), _p(ctx.seg_starts), _p(ctx.seg_slots), _p(state), stride, T, H, G, N, P, taps, _dt(out), _stream()), "ssd_gate")
+                         _p(ctx.seg_starts), _p(ctx.seg_slots), ctx.num_segments, _p(state), stride, T, H, G, N, P, taps, _dt(out), _stream()), "ssd_gate")
     return out
