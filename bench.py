@@ -30,6 +30,9 @@ weights: the same measurements as --workload lupanex (SIPARAX_SIZES below).
 --workload tinevik: the Tinevik design (gated linear attention, attention with capped and mixed scores and rotated values, windowed
 latent attention, experts chosen by a table) beside Manatar with routed feed-forwards at equal width, depth, heads and weights a
 token uses: the same measurements (TINEVIK_SIZES below).
+--workload lirutar: the Lirutar design (attention over a window and a state-space mixer side by side in every layer, looped layers,
+experts chosen by corrected scores inside groups) beside Tinevik at equal width, runs of a layer, heads and feed-forward weights a token
+uses: the same measurements (LIRUTAR_SIZES below).
 --workload prefill8k: one 8,192-token prompt, in one step and in portions of 2,048 through the scheduler.
 
 --impl reference builds nothing of this repository's engine: it runs the unmodified reference program
