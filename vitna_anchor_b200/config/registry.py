@@ -78,3 +78,7 @@ def _register_builtin() -> None:
     from . import lirutar as _lrc
     register_architecture(Architecture(_lrc.ARCHITECTURE, _lrc.LirutarConfig.from_dict, _lr.lirutar_manifest, _lr.build_lirutar,
                                        _lr.is_norm_weight), replace=True)
+    from ..models import zolapel as _zl
+    from . import zolapel as _zlc
+    register_architecture(Architecture(_zlc.ARCHITECTURE, _zlc.ZolapelConfig.from_dict, _zl.zolapel_manifest, _zl.build_zolapel,
+                                       _zl.is_norm_weight), replace=True)

@@ -46,7 +46,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 2) attention_decode_kernel(
     const int32_t* __restrict__ token_seg, const int32_t* __restrict__ positions, const int32_t* __restrict__ tok_list,
     T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int nh, int nkv,
     int hd, int page_size, int max_blocks, int max_splits, float scale, int window, int vd, const float* __restrict__ dist_bias,
-    int max_dist, int v_in_key, int v_share, int out_ld) {
+    int max_dist, int v_in_key, int v_share, int out_ld, const float* __restrict__ gate, int gate_ld) {
     constexpr int V = Vec16<T>::N;
     extern __shared__ float smem[];
     const int g = nh / nkv;
@@ -248,7 +248,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 2) attention_decode_kernel(
         for (int d = tid; d < vd; d += DEC_THREADS) {
             float o = 0.0f;
             for (int gi = 0; gi < parts; gi++) o += red[gi * vd + d];
-            if (single) out[(size_t)t * out_ld + (size_t)(h0 + h) * vd + d] = from_f32<T>(o * (1.0f / stat_l[h]));
+            if (single) out[(size_t)t * out_ld + (size_t)(h0 + h) * vd + d] = from_f32<T>(gated(o * (1.0f / stat_l[h]), gate, gate_ld, t, h0 + h));
             else part_o[(((size_t)zi * nh + h0 + h) * max_splits + split) * vd + d] = o;
         }
     }
@@ -307,7 +307,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 2) attention_decode_kernel(
             o += a3 * wsp[h * DEC_SPLIT + j + 3];
         }
         for (; j < n_active; j++) o += __ldcg(po + (size_t)j * vd) * wsp[h * DEC_SPLIT + j];
-        out[(size_t)t * out_ld + (size_t)(h0 + h) * vd + d] = from_f32<T>(o * stat_l[h]);
+        out[(size_t)t * out_ld + (size_t)(h0 + h) * vd + d] = from_f32<T>(gated(o * stat_l[h], gate, gate_ld, t, h0 + h));
     }
 }
 
@@ -320,7 +320,7 @@ int launch_decode_mma(const void* q, const void* cache, const int32_t* bt, const
 int launch_decode_mma_values(const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
                              const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
                              int hd, int vd, int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
-                             int out_ld, int v_in_key, int v_share, cudaStream_t stream);
+                             int out_ld, int v_in_key, int v_share, const float* gate, int gate_ld, cudaStream_t stream);
 
 // attention_decode_tma.cu: the persistent kernel for large launches (bfloat16, head size 64).
 bool decode_tma_takes(int n_tokens, int nh, int nkv, int hd, int page_size, int pages, int grid_splits, const void* q, const void* cache,
@@ -389,7 +389,7 @@ VK_API int vk_attention_decode(const void* q, const void* cache, const int32_t* 
         }                                                                                                                            \
         return launch_dependent(kern, grid, dim3(DEC_THREADS), smem, stream, (const T*)q, (const T*)cache, block_tables, token_seg, \
                                 positions, tok_list, (T*)out, part_o, part_ml, counters, nh, nkv, hd, page_size, max_blocks, splits, \
-                                scale, window, hd, (const float*)nullptr, 0, 0, 1, nh * hd);                                         \
+                                scale, window, hd, (const float*)nullptr, 0, 0, 1, nh * hd, (const float*)nullptr, 0);               \
     }
     if (dtype == 0) {
         if (async) GO(float, true) else GO(float, false)
@@ -404,12 +404,13 @@ VK_API int vk_attention_decode(const void* q, const void* cache, const int32_t* 
 // vk_attention_decode_scratch_bytes(tokens, nh, nkv, max(hd, vd), max_context) bytes) and an optional bias by distance.
 // v_in_key: the cache holds keys alone and a key's first vd values are its value (vd <= hd).  Rows of out are out_ld elements apart.
 // v_share > 1: key heads v_share*j .. v_share*j + v_share-1 read value head j (a page holds nkv / v_share heads of values).
-// Always the CUDA-core kernel, in both dtypes.
+// gate float32 [all tokens][gate_ld] or null: head h of token t times sigmoid(gate[t][h]).  bfloat16 without a bias by distance takes the tensor-core
+// form for the sizes it is built for; everything else the CUDA-core kernel.
 VK_API int vk_attention_decode_biased(const void* q, const void* cache, const int32_t* block_tables, const int32_t* token_seg,
                                       const int32_t* positions, const int32_t* tok_list, void* out, void* scratch, int scratch_tokens,
                                       int n_tokens, int nh, int nkv, int hd, int vd, int page_size, int max_blocks, int max_context,
                                       int grid_context, float scale, int window, const float* dist_bias, int max_dist, int v_in_key,
-                                      int v_share, int out_ld, int dtype, cudaStream_t stream) {
+                                      int v_share, int out_ld, const float* gate, int gate_ld, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return VK_OK;
     if (out_ld < nh * vd) return VK_BAD_SHAPE;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || hd <= 0 || vd <= 0 || page_size <= 0 || max_blocks <= 0 || window < 0 || max_context <= 0 ||
@@ -433,7 +434,7 @@ VK_API int vk_attention_decode_biased(const void* q, const void* cache, const in
     auto built = [](int n) { return n == 32 || n == 64 || n == 96 || n == 128; };
     if (dtype == 1 && !dist_bias && built(hd) && built(vd) && ((uintptr_t)q % 16 == 0) && scale > 0.0f)
         return launch_decode_mma_values(q, cache, block_tables, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, hd,
-                                        vd, page_size, max_blocks, splits, grid_splits, tiles, scale, window, out_ld, v_in_key, v_share, stream);
+                                        vd, page_size, max_blocks, splits, grid_splits, tiles, scale, window, out_ld, v_in_key, v_share, gate, gate_ld, stream);
     const size_t smem_base = (size_t)(DEC_G_TILE * hd + DEC_G_TILE * DEC_SPLIT + DEC_THREADS * vec) * sizeof(float);
     const size_t smem_async = smem_base + (size_t)DEC_SPLIT * (hd + vd + 2 * vec) * (dtype == 0 ? 4 : 2);
     const bool async = smem_async <= 100 * 1024;        // two blocks a multiprocessor
@@ -448,7 +449,7 @@ VK_API int vk_attention_decode_biased(const void* q, const void* cache, const in
         }                                                                                                                            \
         return launch_dependent(kern, grid, dim3(DEC_THREADS), smem, stream, (const T*)q, (const T*)cache, block_tables, token_seg, \
                                 positions, tok_list, (T*)out, part_o, part_ml, counters, nh, nkv, hd, page_size, max_blocks, splits, \
-                                scale, window, vd, dist_bias, max_dist, v_in_key, v_share, out_ld);                                  \
+                                scale, window, vd, dist_bias, max_dist, v_in_key, v_share, out_ld, gate, gate_ld);                   \
     }
     if (dtype == 0) {
         if (async) GO(float, true) else GO(float, false)
@@ -527,7 +528,7 @@ VK_API int vk_attention_decode_static(const void* q, const void* cache, const in
         }                                                                                                                     \
         kern<<<grid, DEC_THREADS, smem, stream>>>((const T*)q, (const T*)cache, block_tables, token_seg, positions, tok_list, \
                                                   (T*)out, part_o, part_ml, counters, nh, nkv, hd, page_size, max_blocks,     \
-                                                  splits, scale, window, hd, (const float*)nullptr, 0, 0, 1, nh * hd);        \
+                                                  splits, scale, window, hd, (const float*)nullptr, 0, 0, 1, nh * hd, (const float*)nullptr, 0); \
     }
     if (dtype == 0) {
         if (async) GO(float, true) else GO(float, false)

@@ -71,6 +71,8 @@ struct DmArgs {
     int window;
     int out_ld;                             // elements between rows of out
     int v_in_key, v_share;
+    const float* gate;                      // float32 [tokens][gate_ld]: head h of token t times sigmoid(gate[t][h]); null: no gate
+    int gate_ld;
 };
 
 __device__ __forceinline__ DmItem dm_item(const DmArgs& a, int zi, int y, int split) {
@@ -500,7 +502,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD + VD <= 128 ? 3 : 1) attention_
             acc += reinterpret_cast<const float*>(wo_base + w * 32 * WO_LD)[row * VD + d] * e;
         }
         if (single) {
-            a.out[(size_t)t * a.out_ld + (h0 + row) * VD + d] = __float2bfloat16_rn(acc / l);
+            a.out[(size_t)t * a.out_ld + (h0 + row) * VD + d] = __float2bfloat16_rn(gated(acc / l, a.gate, a.gate_ld, t, h0 + row));
         } else {
             a.part_o[(((size_t)zi * nh + h0 + row) * max_splits + split) * VD + d] = acc;
             if (d == 0) *reinterpret_cast<float2*>(a.part_ml + (((size_t)zi * nh + h0 + row) * max_splits + split) * 2) = make_float2(m, l);
@@ -554,7 +556,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD + VD <= 128 ? 3 : 1) attention_
             }
             mm = cm;
         }
-        a.out[(size_t)t * a.out_ld + (h0 + h) * VD + d] = __float2bfloat16_rn(o / l);
+        a.out[(size_t)t * a.out_ld + (h0 + h) * VD + d] = __float2bfloat16_rn(gated(o / l, a.gate, a.gate_ld, t, h0 + h));
     }
 }
 
@@ -562,12 +564,12 @@ template <int HD, int VD>
 static int launch_dm(const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
                      const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
                      int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
-                     int out_ld, int v_in_key, int v_share, cudaStream_t stream) {
+                     int out_ld, int v_in_key, int v_share, const float* gate, int gate_ld, cudaStream_t stream) {
     const int g = nh / nkv, tiles = nkv * ((g + DM_ROWS - 1) / DM_ROWS);
     int shift = -1;
     for (int b = 0; b < 30; b++) if ((1 << b) == page_size) shift = b;
     DmArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, token_seg, positions, tok_list, (__nv_bfloat16*)out, part_o,
-             part_ml, counters, nh, nkv, page_size, shift, max_blocks, splits, counter_tiles, scale, window, out_ld, v_in_key, v_share};
+             part_ml, counters, nh, nkv, page_size, shift, max_blocks, splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, gate, gate_ld};
     // Three blocks a multiprocessor pay when there are several waves of blocks; with a single wave (a small batch)
     // two blocks and a larger first-level cache were measured faster, so the small launch asks for more shared
     // memory than it uses.
@@ -589,7 +591,7 @@ int launch_decode_mma(const void* q, const void* cache, const int32_t* bt, const
                       cudaStream_t stream) {
 #define GO(HD)                                                                                                                   \
     return launch_dm<HD, HD>(q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
-                         max_blocks, splits, grid_splits, counter_tiles, scale, window, nh * HD, 0, 1, stream)
+                         max_blocks, splits, grid_splits, counter_tiles, scale, window, nh * HD, 0, 1, nullptr, 0, stream)
     switch (hd) {
         case 16: GO(16);
         case 32: GO(32);
@@ -605,10 +607,10 @@ template <int HD>
 static int launch_dm_values(int vd, const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
                             const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
                             int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window, int out_ld,
-                            int v_in_key, int v_share, cudaStream_t stream) {
+                            int v_in_key, int v_share, const float* gate, int gate_ld, cudaStream_t stream) {
 #define GO(VD)                                                                                                                        \
     return launch_dm<HD, VD>(q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
-                             max_blocks, splits, grid_splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, stream)
+                             max_blocks, splits, grid_splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, gate, gate_ld, stream)
     switch (vd) {
         case 32: GO(32);
         case 64: GO(64);
@@ -623,10 +625,10 @@ static int launch_dm_values(int vd, const void* q, const void* cache, const int3
 int launch_decode_mma_values(const void* q, const void* cache, const int32_t* bt, const int32_t* token_seg, const int32_t* positions,
                              const int32_t* tok_list, void* out, float* part_o, float* part_ml, int* counters, int n_tokens, int nh, int nkv,
                              int hd, int vd, int page_size, int max_blocks, int splits, int grid_splits, int counter_tiles, float scale, int window,
-                             int out_ld, int v_in_key, int v_share, cudaStream_t stream) {
+                             int out_ld, int v_in_key, int v_share, const float* gate, int gate_ld, cudaStream_t stream) {
 #define GO(HD)                                                                                                                             \
     return launch_dm_values<HD>(vd, q, cache, bt, token_seg, positions, tok_list, out, part_o, part_ml, counters, n_tokens, nh, nkv, page_size, \
-                                max_blocks, splits, grid_splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, stream)
+                                max_blocks, splits, grid_splits, counter_tiles, scale, window, out_ld, v_in_key, v_share, gate, gate_ld, stream)
     switch (hd) {
         case 32: GO(32);
         case 64: GO(64);

@@ -1,8 +1,9 @@
 // Attention whose heads' scores are capped and mixed before the softmax, over the paged cache, with rotated values.
 //
 //  q, k per head: x / rms(x) * w (one weight for all heads; eps < 0: no norm), then the first `dims` values turned in pairs
-//                 (i, i + dims/2) by p * f_i (f from the host, any rescaling already in it)
-//  v_j            turned over all its pairs (m, m + vdim/2) by j * g_m before it is cached (g null: cached as it is)
+//                 (i, i + dims/2), or (2i, 2i + 1), by p * f_i (f from the host, any rescaling already in it)
+//  v_j            turned over all its pairs (m, m + vdim/2) by j * g_m before it is cached (g null: cached as it is); v_j may be the
+//                 projected key itself, as it is before norm and rotation (v_from_k: the row is [ q | k ])
 //  z_h(i, j)      = scale q_h(i) . k(j), then cap * tanh(z / cap) (cap <= 0: none), then z'_h = sum_g M[h][g] z_g (M null: none)
 //  p_h(i, .)      = softmax of z'_h over the keys j <= i (inside the window, if there is one)
 //  o_h(i)         = sum_j p_h(i, j) v_j, turned back by -i * g_m
@@ -30,7 +31,7 @@ __global__ void __launch_bounds__(256) mixed_attn_prepare_kernel(const float* __
                                                                  const float* __restrict__ kn_w, float eps, const float* __restrict__ freq, int dims,
                                                                  const float* __restrict__ vfreq, T* __restrict__ q_out, T* __restrict__ cache,
                                                                  int nh, int nkv, int hd, int vd, int page_size, const float* __restrict__ bias,
-                                                                 float v_mult) {
+                                                                 float v_mult, int neighbours, int v_from_k) {
     extern __shared__ float mp_turn[];                  // cos and sin of the token's angles: [dims/2][2] for q and k, then [vd/2][2] for v
     dependency_wait();
     let_dependents_start();
@@ -65,16 +66,18 @@ __global__ void __launch_bounds__(256) mixed_attn_prepare_kernel(const float* __
                 inv = 1.0f / sqrtf(ss / (float)hd + eps);
             }
             for (int i = lane; i < half; i += 32) {
+                const int u = neighbours ? 2 * i : i, v2 = neighbours ? 2 * i + 1 : i + half;
                 const float c = mp_turn[2 * i], sn = mp_turn[2 * i + 1];
-                const float a = (at(i) * inv) * (w ? w[i] : 1.0f), b = (at(i + half) * inv) * (w ? w[i + half] : 1.0f);
-                dst[i] = from_f32<T>(a * c - b * sn);
-                dst[i + half] = from_f32<T>(b * c + a * sn);
+                const float a = (at(u) * inv) * (w ? w[u] : 1.0f), b = (at(v2) * inv) * (w ? w[v2] : 1.0f);
+                dst[u] = from_f32<T>(a * c - b * sn);
+                dst[v2] = from_f32<T>(b * c + a * sn);
             }
             for (int d = dims + lane; d < hd; d += 32) dst[d] = from_f32<T>((at(d) * inv) * (w ? w[d] : 1.0f));
         } else if (s >= 0) {                            // a value head
             const int g = h - nh - nkv;
-            const float* v = in + (size_t)(nh + nkv) * hd + (size_t)g * vd;
-            const float* bh = bias ? bias + (size_t)(nh + nkv) * hd + (size_t)g * vd : nullptr;
+            const size_t from = v_from_k ? (size_t)(nh + g) * hd : (size_t)(nh + nkv) * hd + (size_t)g * vd;
+            const float* v = in + from;
+            const float* bh = bias ? bias + from : nullptr;
             auto at = [&](int d) { return (bh ? v[d] + bh[d] : v[d]) * v_mult; };
             T* dst = vbase + ((size_t)g * page_size + off) * vd;
             if (vfreq) {
@@ -180,6 +183,97 @@ __global__ void __launch_bounds__(256) rotary_store_kernel(const float* __restri
             } else {
                 am_store4<T>(dst + 4 * j, v[u]);
             }
+        }
+    }
+}
+
+// mixed_attn_prepare with norms and unturned values, where heads are of an even size up to 256 and everything lies on 8 bytes: a warp takes a
+// head, whose values stay in its registers (up to four pairs a lane) between the sum of squares, the turn and the two stores; a key head
+// whose values are its projected keys writes both from the same registers.  The first head's row is asked for before the angles are
+// worked out.
+template <typename T>
+__global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* __restrict__ proj, int N, const int32_t* __restrict__ positions,
+                                                                  const int32_t* __restrict__ slot, const float* __restrict__ qn_w,
+                                                                  const float* __restrict__ kn_w, float eps, const float* __restrict__ freq, int dims,
+                                                                  T* __restrict__ q_out, T* __restrict__ cache, int nh, int nkv, int hd, int vd, int page_size,
+                                                                  float v_mult, int neighbours, int v_from_k) {
+    extern __shared__ float nr_turn[];                  // [dims/2][2] cos and sin of the token's angles
+    constexpr int P = 4;
+    dependency_wait();
+    let_dependents_start();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const int half = dims / 2, pairs = hd / 2, n_qk = nh + nkv, n_heads = v_from_k ? n_qk : n_qk + nkv;
+    const float* in = proj + (size_t)t * N;
+    const int s = (slot && cache) ? slot[t] : -1;
+    const size_t page_stride = (size_t)nkv * page_size * (hd + vd);
+    T* kbase = s >= 0 ? cache + (size_t)(s / page_size) * page_stride : nullptr;
+    T* vbase = s >= 0 ? kbase + (size_t)nkv * page_size * hd : nullptr;
+    const int off = s >= 0 ? s % page_size : 0;
+    // pair j of a query or key head: the two places that are turned together, or two neighbours behind the turned part
+    auto places = [&](int j, int& a, int& b) {
+        if (!neighbours && j < half) { a = j; b = j + half; } else { a = 2 * j; b = a + 1; }
+    };
+    float2 v[P];
+    auto fetch = [&](int h) {
+        const float* row = in + (size_t)h * hd;
+#pragma unroll
+        for (int p = 0; p < P; p++) {
+            const int j = lane + 32 * p;
+            if (j >= pairs) { v[p] = make_float2(0.0f, 0.0f); continue; }
+            int a, b;
+            places(j, a, b);
+            v[p] = b == a + 1 ? *reinterpret_cast<const float2*>(row + a) : make_float2(row[a], row[b]);
+        }
+    };
+    if (warp < n_qk) fetch(warp);
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float ang = pos * freq[i];
+        nr_turn[2 * i] = cosf(ang);
+        nr_turn[2 * i + 1] = sinf(ang);
+    }
+    __syncthreads();
+    for (int h = warp; h < n_heads; h += nwarps) {
+        if (h >= n_qk) {                                // a value head of its own
+            if (s < 0) continue;
+            const int g = h - n_qk;
+            const float* row = in + (size_t)n_qk * hd + (size_t)g * vd;
+            T* dst = vbase + ((size_t)g * page_size + off) * vd;
+            for (int d = lane; d < vd; d += 32) dst[d] = from_f32<T>(row[d] * v_mult);
+            continue;
+        }
+        if (h != warp) fetch(h);
+        const bool key = h >= nh;
+        if (key && s < 0) continue;
+        const float* w = key ? kn_w : qn_w;
+        T* dst = key ? kbase + ((size_t)(h - nh) * page_size + off) * hd : q_out + ((size_t)t * nh + h) * hd;
+        T* vdst = key && v_from_k ? vbase + ((size_t)(h - nh) * page_size + off) * vd : nullptr;
+        float inv = 1.0f;
+        if (eps >= 0.0f) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int p = 0; p < P; p++) { ss = fmaf(v[p].x, v[p].x, ss); ss = fmaf(v[p].y, v[p].y, ss); }
+            inv = 1.0f / sqrtf(warp_sum(ss) / (float)hd + eps);
+        }
+#pragma unroll
+        for (int p = 0; p < P; p++) {
+            const int j = lane + 32 * p;
+            if (j >= pairs) continue;
+            int a, b;
+            places(j, a, b);
+            if (vdst) {
+                if (b == a + 1) am_store2<T>(vdst + a, v[p].x * v_mult, v[p].y * v_mult);
+                else { vdst[a] = from_f32<T>(v[p].x * v_mult); vdst[b] = from_f32<T>(v[p].y * v_mult); }
+            }
+            float x = v[p].x * inv, y = v[p].y * inv;
+            if (w) { x *= w[a]; y *= w[b]; }
+            if (j < half) {
+                const float c = nr_turn[2 * j], sn = nr_turn[2 * j + 1], u = x * c - y * sn;
+                y = y * c + x * sn;
+                x = u;
+            }
+            if (b == a + 1) am_store2<T>(dst + a, x, y);
+            else { dst[a] = from_f32<T>(x); dst[b] = from_f32<T>(y); }
         }
     }
 }
@@ -704,15 +798,23 @@ using namespace vk;
 // write); qn_w, kn_w float32 [hd] or null; eps < 0: no norm; freq float32 [dims/2] (dims 0: no rotation); vfreq float32 [vd/2] or null.
 VK_API int vk_mixed_attn_prepare(const float* proj, int N, const int32_t* positions, const int32_t* slot, const float* qn_w, const float* kn_w, float eps,
                                  const float* freq, int dims, const float* vfreq, void* q_out, void* cache, int tokens, int nh, int nkv, int hd, int vd,
-                                 int page_size, const float* bias, float v_mult, int dtype, cudaStream_t stream) {
+                                 int page_size, const float* bias, float v_mult, int neighbours, int v_from_k, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
-    if (nh <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || N < (nh + nkv) * hd + nkv * vd || dims < 0 || dims % 2 || dims > hd ||
+    if (nh <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || N < (nh + nkv) * hd + (v_from_k ? 0 : nkv * vd) || (v_from_k && (vd != hd || vfreq)) || dims < 0 || dims % 2 || dims > hd ||
         (dims > 0 && !freq))
         return VK_BAD_SHAPE;
     const size_t smem = (size_t)(dims + vd + 1) * sizeof(float);
     if (smem > 48 * 1024) return VK_TOO_LARGE;
     auto on16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
-    if (eps < 0.0f && !qn_w && !kn_w && !vfreq && hd % 4 == 0 && vd % 4 == 0 && dims % 4 == 0 && N % 4 == 0 && on16(proj) && on16(q_out) && on16(cache) &&
+    auto on8 = [](const void* p) { return ((uintptr_t)p % 8) == 0; };
+    if (!vfreq && !bias && (eps >= 0.0f || neighbours || v_from_k) && hd % 2 == 0 && vd % 2 == 0 && hd <= 256 && N % 2 == 0 && on8(proj) && on8(q_out) && on8(cache)) {
+        if (dtype == 0)
+            return launch_dependent(normed_rotary_store_kernel<float>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
+                                    dims, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size, v_mult, neighbours, v_from_k);
+        return launch_dependent(normed_rotary_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps,
+                                freq, dims, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size, v_mult, neighbours, v_from_k);
+    }
+    if (eps < 0.0f && !neighbours && !v_from_k && !qn_w && !kn_w && !vfreq && hd % 4 == 0 && vd % 4 == 0 && dims % 4 == 0 && N % 4 == 0 && on16(proj) && on16(q_out) && on16(cache) &&
         on16(bias)) {
         if (dtype == 0)
             return launch_dependent(rotary_store_kernel<float>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, freq, dims, (float*)q_out,
@@ -722,9 +824,9 @@ VK_API int vk_mixed_attn_prepare(const float* proj, int N, const int32_t* positi
     }
     if (dtype == 0)
         return launch_dependent(mixed_attn_prepare_kernel<float>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
-                                dims, vfreq, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);
+                                dims, vfreq, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size, bias, v_mult, neighbours, v_from_k);
     return launch_dependent(mixed_attn_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), smem, stream, proj, N, positions, slot, qn_w, kn_w, eps, freq,
-                            dims, vfreq, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size, bias, v_mult);
+                            dims, vfreq, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size, bias, v_mult, neighbours, v_from_k);
 }
 
 VK_API size_t vk_attention_mixed_rows_smem(int nh, int hd, int vd) {

@@ -63,7 +63,8 @@ template <int HD, int VD>
 __global__ void __launch_bounds__(PF_THREADS, pf_blocks(HD, VD)) attention_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache, const int32_t* __restrict__ block_tables,
     const int32_t* __restrict__ tiles, __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int max_blocks, float scale,
-    int window, const float* __restrict__ dist_bias, int max_dist, int v_in_key, int v_share, int out_ld, int page_shift) {
+    int window, const float* __restrict__ dist_bias, int max_dist, int v_in_key, int v_share, int out_ld, int page_shift,
+    const float* __restrict__ gate, int gate_ld) {
     typedef __nv_bfloat16 T;
     constexpr int LD = HD + 8;                      // padded row: 16-byte shifts keep ldmatrix free of bank conflicts
     constexpr int LDV = VD + 8;
@@ -316,7 +317,11 @@ __global__ void __launch_bounds__(PF_THREADS, pf_blocks(HD, VD)) attention_prefi
     }
 
     // ---- normalise and store ---------------------------------------------------------------------------
-    const float inv_a = l_run[0] > 0.0f ? 1.0f / l_run[0] : 0.0f, inv_b = l_run[1] > 0.0f ? 1.0f / l_run[1] : 0.0f;
+    float inv_a = l_run[0] > 0.0f ? 1.0f / l_run[0] : 0.0f, inv_b = l_run[1] > 0.0f ? 1.0f / l_run[1] : 0.0f;
+    if (gate) {
+        if (row_a < rows) inv_a = gated(inv_a, gate, gate_ld, tok0 + row_a, h);
+        if (row_b < rows) inv_b = gated(inv_b, gate, gate_ld, tok0 + row_b, h);
+    }
 #pragma unroll
     for (int i = 0; i < DBLK; i++) {
         const int d = i * 8 + qd * 2;
@@ -330,7 +335,7 @@ __global__ void __launch_bounds__(PF_THREADS, pf_blocks(HD, VD)) attention_prefi
 template <int HD, int VD>
 static int launch_prefill(const void* q, const void* cache, const int32_t* bt, const int32_t* tiles, void* out, int n_tiles, int nh,
                           int nkv, int page_size, int max_blocks, float scale, int window, const float* dist_bias, int max_dist,
-                          int v_in_key, int v_share, int out_ld, cudaStream_t stream) {
+                          int v_in_key, int v_share, int out_ld, const float* gate, int gate_ld, cudaStream_t stream) {
     constexpr int LD = HD + 8, LDV = VD + 8;
     size_t smem = (size_t)(PF_BM * LD + 4 * PF_BN * (LD + LDV)) * 2 + 4 * 128 * sizeof(float);
     const size_t hand = (size_t)(PF_BM * LD + 2 * PF_BN * (LD + LDV)) * 2 + (size_t)PF_GROUP * (VD / 8 * 4 + 4) * sizeof(float);
@@ -344,14 +349,14 @@ static int launch_prefill(const void* q, const void* cache, const int32_t* bt, c
     for (int b = 0; b < 30; b++) if ((1 << b) == page_size) shift = b;
     dim3 grid(n_tiles, nh);
     return launch_plain(kern, grid, dim3(PF_THREADS), smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, tiles,
-                            (__nv_bfloat16*)out, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, shift);
+                            (__nv_bfloat16*)out, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, shift, gate, gate_ld);
 }
 
 template <int HD>
 static int launch_prefill_v(int vd, const void* q, const void* cache, const int32_t* bt, const int32_t* tiles, void* out, int n_tiles, int nh,
                             int nkv, int page_size, int max_blocks, float scale, int window, const float* dist_bias, int max_dist,
-                            int v_in_key, int v_share, int out_ld, cudaStream_t stream) {
-#define GO(VD) return launch_prefill<HD, VD>(q, cache, bt, tiles, out, n_tiles, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, stream)
+                            int v_in_key, int v_share, int out_ld, const float* gate, int gate_ld, cudaStream_t stream) {
+#define GO(VD) return launch_prefill<HD, VD>(q, cache, bt, tiles, out, n_tiles, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, gate, gate_ld, stream)
     switch (vd) {
         case 32: GO(32);
         case 64: GO(64);
@@ -375,7 +380,7 @@ VK_API int vk_attention_prefill(const void* q, const void* cache, const int32_t*
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || max_blocks <= 0 || window < 0) return VK_BAD_SHAPE;
     if (nh > 65535) return VK_TOO_LARGE;
     if (((uintptr_t)q % 16) || ((uintptr_t)cache % 16) || ((uintptr_t)out % 4)) return VK_BAD_ALIGNMENT;
-#define GO(HD) return launch_prefill<HD, HD>(q, cache, block_tables, tiles, out, n_tiles, nh, nkv, page_size, max_blocks, scale, window, nullptr, 0, 0, 1, nh * HD, stream)
+#define GO(HD) return launch_prefill<HD, HD>(q, cache, block_tables, tiles, out, n_tiles, nh, nkv, page_size, max_blocks, scale, window, nullptr, 0, 0, 1, nh * HD, nullptr, 0, stream)
     switch (hd) {
         case 16: GO(16);
         case 32: GO(32);
@@ -391,17 +396,17 @@ VK_API int vk_attention_prefill(const void* q, const void* cache, const int32_t*
 // its values) and an optional bias by distance.  Head sizes 32, 64, 96 and 128 for keys and for values, in any pairing.
 // v_in_key: the cache holds keys alone and a key's first vd values are its value (vd <= hd).
 // v_share > 1: key heads v_share*j .. v_share*j + v_share-1 read value head j (a page holds nkv / v_share heads of values).
-// Rows of out are out_ld elements apart.
+// Rows of out are out_ld elements apart.  gate float32 [all tokens][gate_ld] or null: head h of token t times sigmoid(gate[t][h]).
 VK_API int vk_attention_prefill_biased(const void* q, const void* cache, const int32_t* block_tables, const int32_t* tiles, void* out,
                                        int n_tiles, int nh, int nkv, int hd, int vd, int page_size, int max_blocks, float scale, int window,
-                                       const float* dist_bias, int max_dist, int v_in_key, int v_share, int out_ld, cudaStream_t stream) {
+                                       const float* dist_bias, int max_dist, int v_in_key, int v_share, int out_ld, const float* gate, int gate_ld, cudaStream_t stream) {
     if (n_tiles <= 0) return VK_OK;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || max_blocks <= 0 || window < 0 || (dist_bias && max_dist <= 0)) return VK_BAD_SHAPE;
     if ((v_in_key && vd > hd) || out_ld < nh * vd || out_ld % 2) return VK_BAD_SHAPE;
     if (v_share < 1 || nkv % v_share != 0 || (v_in_key && v_share != 1)) return VK_BAD_SHAPE;
     if (nh > 65535) return VK_TOO_LARGE;
     if (((uintptr_t)q % 16) || ((uintptr_t)cache % 16) || ((uintptr_t)out % 4)) return VK_BAD_ALIGNMENT;
-#define GO(HD) return launch_prefill_v<HD>(vd, q, cache, block_tables, tiles, out, n_tiles, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, stream)
+#define GO(HD) return launch_prefill_v<HD>(vd, q, cache, block_tables, tiles, out, n_tiles, nh, nkv, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, gate, gate_ld, stream)
     switch (hd) {
         case 32: GO(32);
         case 64: GO(64);

@@ -18,7 +18,8 @@
 // Two things beyond the plain form, both optional: values of another size than the keys (vd != hd; a page then
 // holds [nkv][page_size][hd] keys followed by [nkv][page_size][vd] values, which for vd == hd is the usual
 // [2][nkv][page_size][hd]), and a bias that depends on the distance between query and key, added to the scaled
-// score: dist_bias [max_dist][nh] float32, row min(pos - key, max_dist - 1).
+// score: dist_bias [max_dist][nh] float32, row min(pos - key, max_dist - 1).  A head's output may be multiplied by the sigmoid of one
+// number a token and head (gate).
 #include "common.cuh"
 
 namespace vk {
@@ -31,7 +32,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attention_rows_kernel(
     const T* __restrict__ q, const T* __restrict__ cache, const int32_t* __restrict__ block_tables,
     const int32_t* __restrict__ token_seg, const int32_t* __restrict__ positions, const int32_t* __restrict__ tok_list,
     T* __restrict__ out, int nh, int nkv, int hd, int vd, int page_size, int max_blocks, float scale, int window,
-    const float* __restrict__ dist_bias, int max_dist, int v_in_key, int v_share, int out_ld) {
+    const float* __restrict__ dist_bias, int max_dist, int v_in_key, int v_share, int out_ld, const float* __restrict__ gate, int gate_ld) {
     extern __shared__ float smem[];
     float* qs = smem;                         // [hd]
     float* pr = qs + hd;                      // [128]
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attention_rows_kernel(
 #pragma unroll
     for (int a = 0; a < ATT_MAX_ACC; a++) {
         const int d = tid + a * ATT_THREADS;
-        if (d < vd) orow[d] = from_f32<T>(acc[a] * inv);
+        if (d < vd) orow[d] = from_f32<T>(gated(acc[a] * inv, gate, gate_ld, t, h));
     }
 }
 
@@ -111,11 +112,12 @@ using namespace vk;
 // block_tables [segments, max_blocks]; token_seg, positions [all tokens]; tok_list [tokens] names the
 // tokens to run (null: 0..tokens-1); dist_bias [max_dist][nh] float32 or null.  v_share > 1: key heads v_share*j .. v_share*j + v_share-1 read value
 // head j, and a page holds [nkv][page_size][hd] keys followed by [nkv / v_share][page_size][vd] values.  v_in_key: the cache holds keys alone,
-// [pages][nkv*page_size*hd], and a key's first vd values are its value (vd <= hd).
+// [pages][nkv*page_size*hd], and a key's first vd values are its value (vd <= hd).  gate float32 [all tokens][gate_ld] or null: head h of
+// token t times sigmoid(gate[t][h]).
 VK_API int vk_attention_rows_biased(const void* q, const void* cache, const int32_t* block_tables, const int32_t* token_seg,
                                     const int32_t* positions, const int32_t* tok_list, void* out, int tokens, int nh, int nkv, int hd, int vd,
                                     int page_size, int max_blocks, float scale, int window, const float* dist_bias, int max_dist, int v_in_key,
-                                    int v_share, int out_ld, int dtype, cudaStream_t stream) {
+                                    int v_share, int out_ld, const float* gate, int gate_ld, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || hd <= 0 || vd <= 0 || page_size <= 0 || max_blocks <= 0 || window < 0) return VK_BAD_SHAPE;
     if (dist_bias && max_dist <= 0) return VK_BAD_SHAPE;
@@ -129,11 +131,11 @@ VK_API int vk_attention_rows_biased(const void* q, const void* cache, const int3
     if (dtype == 0)
         attention_rows_kernel<float><<<grid, ATT_THREADS, smem, stream>>>((const float*)q, (const float*)cache, block_tables,
                                                                           token_seg, positions, tok_list, (float*)out, nh, nkv, hd, vd,
-                                                                          page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld);
+                                                                          page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, gate, gate_ld);
     else
         attention_rows_kernel<__nv_bfloat16><<<grid, ATT_THREADS, smem, stream>>>(
             (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, token_seg, positions, tok_list, (__nv_bfloat16*)out, nh,
-            nkv, hd, vd, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld);
+            nkv, hd, vd, page_size, max_blocks, scale, window, dist_bias, max_dist, v_in_key, v_share, out_ld, gate, gate_ld);
     return launch_status();
 }
 
@@ -143,5 +145,5 @@ VK_API int vk_attention_rows(const void* q, const void* cache, const int32_t* bl
                              int max_blocks, float scale, int window, int dtype, cudaStream_t stream) {
     if (hd > ATT_THREADS * ATT_MAX_ACC) return VK_TOO_LARGE;
     return vk_attention_rows_biased(q, cache, block_tables, token_seg, positions, tok_list, out, tokens, nh, nkv, hd, hd, page_size, max_blocks,
-                                    scale, window, nullptr, 0, 0, 1, nh * hd, dtype, stream);
+                                    scale, window, nullptr, 0, 0, 1, nh * hd, nullptr, 0, dtype, stream);
 }

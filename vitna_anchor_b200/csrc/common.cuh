@@ -101,6 +101,12 @@ __device__ __forceinline__ float activate_dense(int kind, float z) {
     return activate_rt(kind, z);
 }
 
+// What a head's output is multiplied by where an attention has a gate a head: the sigmoid of the token's number for the head, gate float32
+// [tokens][ld] (null: nothing is multiplied).
+__device__ __forceinline__ float gated(float v, const float* __restrict__ gate, int ld, int t, int h) {
+    return gate ? v * (1.0f / (1.0f + expf(-gate[(size_t)t * ld + h]))) : v;
+}
+
 inline int launch_status() { return (int)cudaGetLastError(); }
 
 // Programmatic dependent launch.  A kernel launched with launch_dependent() may start while the kernel before it

@@ -1,14 +1,17 @@
-// A routed feed-forward: every token uses `top` of E small gated feed-forward layers, weighted by a softmax over the chosen logits.
+// A routed feed-forward: every token uses `top` of E small feed-forward layers (gated or not), with weights from a router or a table.
 //
 //  experts_route     one block a token: logits z = W_r x + b in float32 (a warp a logit), the `top` largest (of equal logits the lower
 //                    index), weights = softmax over the chosen logits alone.  Writes ids [tokens][top] and weights [tokens][top].
 //  experts_route_scored  scores s = softmax(W_r x) over experts AND identities; a token's choice goes by s + correction: of `count` equal
 //                    groups of neighbours only the `keep` with the largest choice score take part, and of their members the `top` with the
 //                    largest (of equals the lower index); weights s / (sum of the chosen s + 1e-20) times scale.  An id of E or more
-//                    is an identity: its output is the token's input row.
+//                    is an identity: its output is the token's input row.  The other form has a sigmoid for every score and takes the
+//                    chosen scores as they are, times scale (without a correction the logits choose: a sigmoid that has rounded
+//                    to 1 does not make a tie); squared, if asked: where the weight multiplies the INPUT of an expert whose
+//                    activation is homogeneous of degree 2, f(s z) = s^2 f(z), its square multiplies the output.
 //  experts_route_table  ids[token][k] = table[token id][k], every weight 1 / top: the experts of a token are a function of its id.
 //  experts_gate_up   act[token, k] = f(W_gate,e x) * (W_up,e x) for the token's k-th expert e; a warp an output column, the token's row
-//                    in shared memory.  f is one of the epilogues' activations.
+//                    in shared memory.  f is one of the epilogues' activations.  Ungated: act[token, k] = f(W_up,e x).
 //  experts_down      y[token] += sum_k weight_k W_down,e_k act[token, k], the experts of a token summed in the order of its list, so
 //                    that the sum does not depend on what else is in the batch.
 //
@@ -81,7 +84,8 @@ __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict_
 template <typename T, int TB>
 __global__ void __launch_bounds__(256) experts_route_scored_kernel(const T* __restrict__ x, int width, const float* __restrict__ wr,
                                                                    const float* __restrict__ correction, int all, int top, int count, int keep, float scale,
-                                                                   int32_t* __restrict__ ids, float* __restrict__ wts, int tokens, int vec) {
+                                                                   int32_t* __restrict__ ids, float* __restrict__ wts, int tokens, int vec, int sigmoid,
+                                                                   int squared) {
     extern __shared__ float rs_sm[];                    // [TB][all] scores | [TB][all] choice scores | [TB][count] the groups' best
     dependency_wait();
     let_dependents_start();
@@ -125,15 +129,23 @@ __global__ void __launch_bounds__(256) experts_route_scored_kernel(const T* __re
     float* s = rs_sm + warp * all;
     float* choice = rs_sm + TB * all + warp * all;
     float* best_of = rs_sm + 2 * TB * all + warp * count;
-    float mx = -INFINITY, sum = 0.0f;
-    for (int e = lane; e < all; e += 32) mx = fmaxf(mx, s[e]);
-    mx = warp_max(mx);
-    for (int e = lane; e < all; e += 32) { const float v = expf(s[e] - mx); s[e] = v; sum += v; }
-    sum = warp_sum(sum);
-    for (int e = lane; e < all; e += 32) {
-        const float v = s[e] / sum;
-        s[e] = v;
-        choice[e] = v + (correction ? correction[e] : 0.0f);
+    if (sigmoid) {
+        for (int e = lane; e < all; e += 32) {
+            const float z = s[e], v = 1.0f / (1.0f + expf(-z));
+            s[e] = v;
+            choice[e] = correction ? v + correction[e] : z;
+        }
+    } else {
+        float mx = -INFINITY, sum = 0.0f;
+        for (int e = lane; e < all; e += 32) mx = fmaxf(mx, s[e]);
+        mx = warp_max(mx);
+        for (int e = lane; e < all; e += 32) { const float v = expf(s[e] - mx); s[e] = v; sum += v; }
+        sum = warp_sum(sum);
+        for (int e = lane; e < all; e += 32) {
+            const float v = s[e] / sum;
+            s[e] = v;
+            choice[e] = v + (correction ? correction[e] : 0.0f);
+        }
     }
     __syncwarp();
     // the largest of n values (of equals the first), which then counts no more; every lane gets its index
@@ -174,7 +186,8 @@ __global__ void __launch_bounds__(256) experts_route_scored_kernel(const T* __re
     }
     if (lane < top) {
         ids[(size_t)t * top + lane] = id;
-        wts[(size_t)t * top + lane] = mine / (chosen + 1e-20f) * scale;
+        const float w = sigmoid ? mine * scale : mine / (chosen + 1e-20f) * scale;
+        wts[(size_t)t * top + lane] = squared ? w * w : w;
     }
 }
 
@@ -192,8 +205,8 @@ __global__ void __launch_bounds__(256) experts_route_table_kernel(const int32_t*
     wts[i] = 1.0f / (float)top;
 }
 
-// grid (pairs, column groups); a warp a column
-template <typename T>
+// grid (pairs, column groups); a warp a column.  wgu [E][2 ff][width] (a group's gate rows, then its up rows), or [E][ff][width] ungated
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restrict__ x, int width, const T* __restrict__ wgu, int ff, int top,
                                                               const int32_t* __restrict__ ids, int E, int act, float limit, float alpha,
                                                               T* __restrict__ out, int vec) {
@@ -206,7 +219,7 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
     if (e >= E) return;                                 // an identity
     for (int i = threadIdx.x; i < width; i += blockDim.x) xs[i] = to_f32<T>(x[(size_t)t * width + i]);
     __syncthreads();
-    const T* wg = wgu + (size_t)e * 2 * ff * width;
+    const T* wg = wgu + (size_t)e * (GATED ? 2 : 1) * ff * width;
     const T* wu = wg + (size_t)ff * width;
     for (int c = blockIdx.y * nwarps + warp; c < ff; c += gridDim.y * nwarps) {
         const T* g = wg + (size_t)c * width;
@@ -218,25 +231,27 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
             for (int i = lane * V; i < width; i += 32 * V) {
                 float gv[V], uv[V];
                 load16<T>(g + i, gv);
-                load16<T>(u + i, uv);
+                if (GATED) load16<T>(u + i, uv);
 #pragma unroll
                 for (int e = 0; e < V; e += 4) {
                     const float4 x4 = *reinterpret_cast<const float4*>(xs + i + e);
                     ag = fmaf(x4.x, gv[e], ag); ag = fmaf(x4.y, gv[e + 1], ag); ag = fmaf(x4.z, gv[e + 2], ag); ag = fmaf(x4.w, gv[e + 3], ag);
-                    au = fmaf(x4.x, uv[e], au); au = fmaf(x4.y, uv[e + 1], au); au = fmaf(x4.z, uv[e + 2], au); au = fmaf(x4.w, uv[e + 3], au);
+                    if (GATED) { au = fmaf(x4.x, uv[e], au); au = fmaf(x4.y, uv[e + 1], au); au = fmaf(x4.z, uv[e + 2], au); au = fmaf(x4.w, uv[e + 3], au); }
                 }
             }
         } else {
             for (int i = lane; i < width; i += 32) {
                 ag = fmaf(xs[i], to_f32<T>(g[i]), ag);
-                au = fmaf(xs[i], to_f32<T>(u[i]), au);
+                if (GATED) au = fmaf(xs[i], to_f32<T>(u[i]), au);
             }
         }
         ag = warp_sum(ag);
-        au = warp_sum(au);
+        if (GATED) au = warp_sum(au);
         if (lane == 0) {
             float r;
-            if (act == 4) {                             // the clamped form: min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + 1)
+            if (!GATED) {
+                r = activate_dense(act, ag);
+            } else if (act == 4) {                             // the clamped form: min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + 1)
                 const float g = fminf(ag, limit), u = fminf(fmaxf(au, -limit), limit);
                 r = (g / (1.0f + expf(-alpha * g))) * (u + 1.0f);
             } else {
@@ -433,9 +448,10 @@ VK_API int vk_experts_combine(const float* o, int width, int top, const int32_t*
 }
 
 // x [tokens][width] in dtype; wr float32 [all][width], correction float32 [all] or null, all = experts + identities, in `count` equal groups of
-// neighbours of which `keep` take part; ids int32 [tokens][top], wts float32 [tokens][top].
+// neighbours of which `keep` take part; ids int32 [tokens][top], wts float32 [tokens][top].  sigmoid 1: the form with a sigmoid a score;
+// squared 1: the weights' squares.
 VK_API int vk_experts_route_scored(const void* x, int width, const float* wr, const float* correction, int all, int top, int count, int keep, float scale,
-                                   int32_t* ids, float* wts, int tokens, int dtype, cudaStream_t stream) {
+                                   int sigmoid, int squared, int32_t* ids, float* wts, int tokens, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
     if (width <= 0 || all <= 0 || count <= 0 || all % count || keep <= 0 || keep > count || top <= 0 || top > 32 || top > all / count * keep) return VK_BAD_SHAPE;
     const int tb = tokens > 64 ? 4 : 1;
@@ -445,7 +461,7 @@ VK_API int vk_experts_route_scored(const void* x, int width, const float* wr, co
     const int vec = width % (dtype == 0 ? 4 : 8) == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)wr % 16) == 0;
 #define VK_ERS(T, TB)                                                                                                                          \
     return launch_dependent(experts_route_scored_kernel<T, TB>, grid, dim3(256), smem, stream, (const T*)x, width, wr, correction, all, top, count, \
-                            keep, scale, ids, wts, tokens, vec)
+                            keep, scale, ids, wts, tokens, vec, sigmoid, squared)
     if (dtype == 0) {
         if (tb == 4) VK_ERS(float, 4);
         VK_ERS(float, 1);
@@ -478,21 +494,26 @@ VK_API int vk_experts_route_table(const int32_t* tokens, const int32_t* table, i
 
 // wgu [E][2 ff][width] (an expert's gate rows, then its up rows) in dtype; out [tokens * top][ff] in dtype.  act: 0 none, 1 gelu (erf),
 // 2 gelu (tanh), 3 silu, 4 the clamped form min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).
-VK_API int vk_experts_gate_up(const void* x, int width, const void* wgu, int ff, int top, const int32_t* ids, int E, int act, float limit, float alpha,
-                              void* out, int tokens, int dtype, cudaStream_t stream) {
+// gated 0: wgu [E][ff][width], and act as activate_dense numbers them (4 is relu squared).
+VK_API int vk_experts_gate_up(const void* x, int width, const void* wgu, int ff, int top, const int32_t* ids, int E, int gated, int act, float limit,
+                              float alpha, void* out, int tokens, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
-    if (width <= 0 || ff <= 0 || top <= 0 || act < 0 || act > 4 || (act == 4 && !(limit > 0.0f))) return VK_BAD_SHAPE;
+    if (width <= 0 || ff <= 0 || top <= 0 || act < 0 || act > 4 || (gated && act == 4 && !(limit > 0.0f))) return VK_BAD_SHAPE;
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 48 * 1024) return VK_TOO_LARGE;
     int gy = (ff + 7) / 8;
     if (gy > 64) gy = 64;
     dim3 grid(tokens * top, gy);
     const int vec = width % (dtype == 0 ? 4 : 8) == 0 && ((uintptr_t)wgu % 16) == 0;
-    if (dtype == 0)
-        return launch_dependent(experts_gate_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, width, (const float*)wgu, ff, top, ids, E, act,
-                                limit, alpha, (float*)out, vec);
-    return launch_dependent(experts_gate_up_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, width,
-                            (const __nv_bfloat16*)wgu, ff, top, ids, E, act, limit, alpha, (__nv_bfloat16*)out, vec);
+    auto go = [&](auto kf, auto kb) {
+        if (dtype == 0)
+            return launch_dependent(kf, grid, dim3(256), smem, stream, (const float*)x, width, (const float*)wgu, ff, top, ids, E, act, limit, alpha,
+                                    (float*)out, vec);
+        return launch_dependent(kb, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, width, (const __nv_bfloat16*)wgu, ff, top, ids, E, act, limit,
+                                alpha, (__nv_bfloat16*)out, vec);
+    };
+    if (gated) return go(experts_gate_up_kernel<float, true>, experts_gate_up_kernel<__nv_bfloat16, true>);
+    return go(experts_gate_up_kernel<float, false>, experts_gate_up_kernel<__nv_bfloat16, false>);
 }
 
 // act [tokens * top][ff] and wd [E][width][ff] in dtype; y float32 [tokens][width] is added to; ids of E and more: the token's row of x.

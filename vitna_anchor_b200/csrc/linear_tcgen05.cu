@@ -856,13 +856,13 @@ static int linear_tcgen05_gated_impl(const void* x, const void* w, void* out, in
 
 // Products of row groups with a weight matrix each.  x [M, K] bfloat16 holds the groups' rows one group after another, every group
 // filled up to whole tiles of 128 rows; tile_group int32 [ceil(M / 128)] on the device names each tile's group (negative: an unused
-// tile).  gated 0: w [groups][N][K], out [M, N] (mode 0 bfloat16, 1 float32) = x w_g^T.  gated 1: w [groups][2 N][K] (a group's gate
+// tile).  gated 0: w [groups][N][K], out [M, N] (mode 0 bfloat16, 1 float32) = x w_g^T, in mode 0 with activate_dense's number act (0: none).  gated 1: w [groups][2 N][K] (a group's gate
 // rows, then its up rows), out [M, N] bfloat16 = f(x gate_g^T) * (x up_g^T), f = silu (act 0) or activate_rt's number act.
 VK_API int vk_linear_tcgen05_grouped(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int groups, const int32_t* tile_group,
                                      int mode, int gated, int act, int* error, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return VK_OK;
-    if (K <= 0 || ldx < K || !error || !tile_group || groups <= 0 || K % 8 != 0 || ldx % 8 != 0 || act < 0 || act > 3) return VK_BAD_SHAPE;
-    if (gated ? (N % 8 != 0 || mode != 0) : (mode < 0 || mode > 1 || act != 0)) return VK_BAD_SHAPE;
+    if (K <= 0 || ldx < K || !error || !tile_group || groups <= 0 || K % 8 != 0 || ldx % 8 != 0 || act < 0 || act > 4) return VK_BAD_SHAPE;
+    if (gated ? (N % 8 != 0 || mode != 0 || act > 3) : (mode < 0 || mode > 1 || (act != 0 && mode != 0))) return VK_BAD_SHAPE;
     if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || ((uintptr_t)out % 16)) return VK_BAD_ALIGNMENT;
     if ((M + TC_BM - 1) / TC_BM > 65535 || (long long)groups * (gated ? 2 : 1) * N > 0x7fffffffLL) return VK_TOO_LARGE;
     CUtensorMap mx, mw;

@@ -794,18 +794,29 @@ def _out_rows(out: torch.Tensor, dtype: torch.dtype, rows: int, width: int, name
     return max(out.stride(0), width)
 
 
+def _gate_rows(gate: Optional[torch.Tensor], rows: int, heads: int, name: str) -> int:
+    """The distance in elements between the rows of an attention's gate, which may be columns of a wider matrix."""
+    if gate is None:
+        return 0
+    if not gate.is_cuda or gate.dtype != torch.float32 or gate.shape != (rows, heads) or gate.stride(1) != 1:
+        raise KernelError(f"{name}: the gate is not a float32 CUDA matrix [tokens, heads] with unit column stride")
+    return max(gate.stride(0), heads)
+
+
 def attention_rows_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_tables: torch.Tensor, token_seg: torch.Tensor,
                           positions: torch.Tensor, out: torch.Tensor, nh: int, nkv: int, hd: int, vd: int, page_size: int, scale: float,
                           window: int = 0, dist_bias: Optional[torch.Tensor] = None, tok_list: Optional[torch.Tensor] = None,
-                          v_in_key: bool = False, v_share: int = 1) -> torch.Tensor:
+                          v_in_key: bool = False, v_share: int = 1, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of every token (or of those in tok_list) over its request's pages, any sizes, float32 arithmetic,
     with values of size vd and, if given, dist_bias [distances, nh] (float32) added to the scaled scores by min(distance, last row).
     v_in_key: the cache holds keys alone and a key's first vd values are its value.  v_share > 1: that many neighbouring
-    key heads read one value head (two score maps over the same values)."""
+    key heads read one value head (two score maps over the same values).  gate float32 [T, nh] (its rows may lie apart): head h of
+    token t is multiplied by sigmoid(gate[t, h])."""
     _req(q, "q", dims=2); _req(cache_layer, "cache_layer", q.dtype); _req(block_tables, "block_tables", torch.int32, 2)
     _req(token_seg, "token_seg", torch.int32, 1); _req(positions, "positions", torch.int32, 1)
     T = q.shape[0]
     out_ld = _out_rows(out, q.dtype, T, nh * vd, "attention_rows_biased")
+    gate_ld = _gate_rows(gate, T, nh, "attention_rows_biased")
     if q.shape[1] != nh * hd or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size:
         raise KernelError("attention_rows_biased: shapes do not fit the head counts")
     if token_seg.shape[0] != T or positions.shape[0] != T:
@@ -820,7 +831,7 @@ def attention_rows_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_tabl
         n = tok_list.shape[0]
     _check(lib().vk_attention_rows_biased(_p(q), _p(cache_layer), _p(block_tables), _p(token_seg), _p(positions), _p(tok_list), _p(out), n, nh,
                                           nkv, hd, vd, page_size, block_tables.shape[1], ctypes.c_float(scale), window, _p(dist_bias),
-                                          0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _dt(q), _stream()),
+                                          0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _p(gate), gate_ld, _dt(q), _stream()),
            "attention_rows_biased")
     return out
 
@@ -904,14 +915,16 @@ def attention_decode_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_ta
                             positions: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, scratch_tokens: int, nh: int, nkv: int, hd: int,
                             vd: int, page_size: int, scale: float, max_context: int, grid_context: int, window: int = 0,
                             dist_bias: Optional[torch.Tensor] = None, tok_list: Optional[torch.Tensor] = None,
-                            v_in_key: bool = False, v_share: int = 1) -> torch.Tensor:
+                            v_in_key: bool = False, v_share: int = 1, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The split-key attention of single decoded tokens in the unrotated form: values of size vd, an optional bias by distance.
-    scratch: attention_decode_scratch_bytes(scratch_tokens, nh, nkv, max(hd, vd), max_context) bytes, zero at first use."""
+    scratch: attention_decode_scratch_bytes(scratch_tokens, nh, nkv, max(hd, vd), max_context) bytes, zero at first use.  gate: as in
+    attention_rows_biased."""
     _req(q, "q", dims=2); _req(cache_layer, "cache_layer", q.dtype); _req(block_tables, "block_tables", torch.int32, 2)
     _req(token_seg, "token_seg", torch.int32, 1); _req(positions, "positions", torch.int32, 1)
     _req(scratch, "scratch", torch.uint8, 1)
     T = q.shape[0]
     out_ld = _out_rows(out, q.dtype, T, nh * vd, "attention_decode_biased")
+    gate_ld = _gate_rows(gate, T, nh, "attention_decode_biased")
     if q.shape[1] != nh * hd or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size:
         raise KernelError("attention_decode_biased: shapes do not fit the head counts")
     if dist_bias is not None:
@@ -927,8 +940,8 @@ def attention_decode_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_ta
     _check(lib().vk_attention_decode_biased(_p(q), _p(cache_layer), _p(block_tables), _p(token_seg), _p(positions), _p(tok_list), _p(out),
                                             _p(scratch), scratch_tokens, n, nh, nkv, hd, vd, page_size, block_tables.shape[1], max_context,
                                             grid_context, ctypes.c_float(scale), window, _p(dist_bias),
-                                            0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _dt(q), _stream()),
-           "attention_decode_biased")
+                                            0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _p(gate), gate_ld,
+                                            _dt(q), _stream()), "attention_decode_biased")
     return out
 
 
@@ -937,12 +950,14 @@ BIASED_PREFILL_HEAD_SIZES = (32, 64, 96, 128)
 
 def attention_prefill_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_tables: torch.Tensor, tiles: torch.Tensor, out: torch.Tensor,
                              nh: int, nkv: int, hd: int, vd: int, page_size: int, scale: float, window: int = 0,
-                             dist_bias: Optional[torch.Tensor] = None, v_in_key: bool = False, v_share: int = 1) -> torch.Tensor:
+                             dist_bias: Optional[torch.Tensor] = None, v_in_key: bool = False, v_share: int = 1,
+                             gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of prompt portions in bfloat16 on the tensor cores, in the unrotated form.  tiles int32 [n, 4]: first
-    token, rows (1..64), position of the first token, segment."""
+    token, rows (1..64), position of the first token, segment.  gate: as in attention_rows_biased."""
     _req(q, "q", torch.bfloat16, 2); _req(cache_layer, "cache_layer", torch.bfloat16)
     _req(block_tables, "block_tables", torch.int32, 2); _req(tiles, "tiles", torch.int32, 2)
     out_ld = _out_rows(out, torch.bfloat16, q.shape[0], nh * vd, "attention_prefill_biased")
+    gate_ld = _gate_rows(gate, q.shape[0], nh, "attention_prefill_biased")
     if (q.shape[1] != nh * hd or _page_size_of(cache_layer, nkv, hd, 0 if v_in_key else vd, v_share) != page_size
             or tiles.shape[1] != 4):
         raise KernelError("attention_prefill_biased: shapes do not fit the head counts")
@@ -954,15 +969,16 @@ def attention_prefill_biased(q: torch.Tensor, cache_layer: torch.Tensor, block_t
             raise KernelError("attention_prefill_biased: the bias table is not [distances, heads]")
     _check(lib().vk_attention_prefill_biased(_p(q), _p(cache_layer), _p(block_tables), _p(tiles), _p(out), tiles.shape[0], nh, nkv, hd, vd,
                                              page_size, block_tables.shape[1], ctypes.c_float(scale), window, _p(dist_bias),
-                                             0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _stream()), "attention_prefill_biased")
+                                             0 if dist_bias is None else dist_bias.shape[0], int(v_in_key), int(v_share), out_ld, _p(gate),
+                                             gate_ld, _stream()), "attention_prefill_biased")
     return out
 
 
 def attention_biased(q: torch.Tensor, pages: torch.Tensor, meta, ctx, out: torch.Tensor, nh: int, nkv: int, hd: int, vd: int,
                      page_size: int, scale: float, window: int = 0, dist_bias: Optional[torch.Tensor] = None,
-                     v_in_key: bool = False, v_share: int = 1) -> torch.Tensor:
+                     v_in_key: bool = False, v_share: int = 1, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of a mixed batch over the paged cache in the unrotated form (values of their own size, or the
-    first vd values of the keys with v_in_key; v_share neighbouring key heads reading one value head; a bias by distance); `meta` is the page group's GroupMeta.  Single decoded tokens take the split-key kernel, tokens of prompt
+    first vd values of the keys with v_in_key; v_share neighbouring key heads reading one value head; a bias by distance; a gate a head); `meta` is the page group's GroupMeta.  Single decoded tokens take the split-key kernel, tokens of prompt
     portions the tensor-core kernel (bfloat16, head sizes it is built for); whatever is left, and the whole exact 32-bit
     routing, takes attention_rows_biased, which takes every size."""
     vec = 4 if q.dtype == torch.float32 else 8
@@ -973,16 +989,17 @@ def attention_biased(q: torch.Tensor, pages: torch.Tensor, meta, ctx, out: torch
               and ctx.pre_tiles is not None and q.data_ptr() % 16 == 0 and pages.data_ptr() % 16 == 0 and out.data_ptr() % 4 == 0
               and out.stride(0) % 2 == 0)
     rows = lambda toks: attention_rows_biased(q, pages, meta.block_tables, ctx.token_seg, ctx.positions, out, nh, nkv, hd, vd, page_size,
-                                              scale, window, dist_bias, toks, v_in_key, v_share)
+                                              scale, window, dist_bias, toks, v_in_key, v_share, gate)
     if dec_ok:
         ws = ctx.workspace
         cap, layout = ws.max_segments, ws.max_context
         nbytes = attention_decode_scratch_bytes(cap, nh, nkv, max(hd, vd), layout)
         scratch = ws.flat(f"att.decb/{nh}/{nkv}/{hd}/{vd}/{layout}", nbytes, torch.uint8, zero=True)
         attention_decode_biased(q, pages, meta.block_tables, ctx.token_seg, ctx.positions, out, scratch, cap, nh, nkv, hd, vd, page_size,
-                                scale, layout, min(layout, max(1, ctx.max_context)), window, dist_bias, ctx.dec_tokens, v_in_key, v_share)
+                                scale, layout, min(layout, max(1, ctx.max_context)), window, dist_bias, ctx.dec_tokens, v_in_key, v_share, gate)
     if pre_ok:
-        attention_prefill_biased(q, pages, meta.block_tables, ctx.pre_tiles, out, nh, nkv, hd, vd, page_size, scale, window, dist_bias, v_in_key, v_share)
+        attention_prefill_biased(q, pages, meta.block_tables, ctx.pre_tiles, out, nh, nkv, hd, vd, page_size, scale, window, dist_bias, v_in_key, v_share,
+                                 gate)
     if not dec_ok and not pre_ok:
         return rows(None)
     if ctx.num_pre and not pre_ok:
@@ -1389,10 +1406,10 @@ def experts_route(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional[to
 
 
 def experts_route_scored(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int, scale: float,
-                         ids: torch.Tensor, wts: torch.Tensor) -> None:
+                         ids: torch.Tensor, wts: torch.Tensor, sigmoid: bool = False, squared: bool = False) -> None:
     """s = softmax(w_router x) over all rows of w_router (experts, then identities); of `groups` equal groups of neighbours the `keep` with the largest
     s + correction; of their members the `top` with the largest s + correction go to ids [T, top], s / (sum of the chosen + 1e-20) * scale to
-    wts [T, top]."""
+    wts [T, top].  sigmoid: s = sigmoid(w_router x), each for itself, and the chosen weights are s * scale.  squared: wts gets the weights' squares."""
     _req(x, "x", dims=2); _req(w_router, "w_router", torch.float32, 2); _req(ids, "ids", torch.int32, 2); _req(wts, "wts", torch.float32, 2)
     T, W = x.shape
     E = w_router.shape[0]
@@ -1400,8 +1417,8 @@ def experts_route_scored(x: torch.Tensor, w_router: torch.Tensor, correction: Op
         raise KernelError("experts_route_scored: shapes do not fit")
     if correction is not None:
         _req(correction, "correction", torch.float32, 1)
-    _check(lib().vk_experts_route_scored(_p(x), W, _p(w_router), _p(correction), E, top, groups, keep, ctypes.c_float(scale), _p(ids), _p(wts), T, _dt(x),
-                                         _stream()), "experts_route_scored")
+    _check(lib().vk_experts_route_scored(_p(x), W, _p(w_router), _p(correction), E, top, groups, keep, ctypes.c_float(scale), int(sigmoid), int(squared),
+                                         _p(ids), _p(wts), T, _dt(x), _stream()), "experts_route_scored")
 
 
 def experts_route_table(tokens: torch.Tensor, table: torch.Tensor, E: int, top: int, ids: torch.Tensor, wts: torch.Tensor) -> None:
@@ -1414,7 +1431,11 @@ def experts_route_table(tokens: torch.Tensor, table: torch.Tensor, E: int, top: 
            "experts_route_table")
 
 
-def _expert_act(activation: str, what: str) -> int:
+def _expert_act(activation: str, what: str, gated: bool = True) -> int:
+    if not gated:
+        if activation not in DENSE_ACTIVATIONS:
+            raise KernelError(f"{what}: {activation!r} is not one of {sorted(DENSE_ACTIVATIONS)}")
+        return DENSE_ACTIVATIONS[activation] + 1
     if activation == "clamped":
         return 4
     if activation not in _EPILOGUE_ACT:
@@ -1423,18 +1444,20 @@ def _expert_act(activation: str, what: str) -> int:
 
 
 def experts_apply(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, act_buf: torch.Tensor,
-                  y: torch.Tensor, activation: str = "silu", limit: float = 0.0, alpha: float = 1.702) -> torch.Tensor:
+                  y: torch.Tensor, activation: str = "silu", limit: float = 0.0, alpha: float = 1.702, gated: bool = True) -> torch.Tensor:
     """y [T, W] (float32) += sum_k wts[t, k] W_down,e (act(W_gate,e x) * W_up,e x), e = ids[t, k] (an id of E or more: x itself); w_gate_up [E, 2 ff, W], w_down [E, W, ff]
-    in x's dtype; act_buf [T * top, ff] in x's dtype.  activation "clamped": min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u) + 1)."""
+    in x's dtype; act_buf [T * top, ff] in x's dtype.  activation "clamped": min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u) + 1).
+    gated False: w_gate_up is [E, ff, W] and an expert W_down,e act(W_up,e x), act one of DENSE_ACTIVATIONS."""
     _req(x, "x", dims=2); _req(w_gate_up, "w_gate_up", x.dtype, 3); _req(w_down, "w_down", x.dtype, 3); _req(y, "y", torch.float32, 2)
     _req(act_buf, "act_buf", x.dtype, 2)
     T, W = x.shape
-    E, two_ff, _ = w_gate_up.shape
-    ff, top = two_ff // 2, ids.shape[1]
-    if w_gate_up.shape != (E, 2 * ff, W) or w_down.shape != (E, W, ff) or y.shape != (T, W) or act_buf.shape != (T * top, ff):
+    E, rows, _ = w_gate_up.shape
+    per = 2 if gated else 1
+    ff, top = rows // per, ids.shape[1]
+    if w_gate_up.shape != (E, per * ff, W) or w_down.shape != (E, W, ff) or y.shape != (T, W) or act_buf.shape != (T * top, ff):
         raise KernelError("experts_apply: shapes do not fit")
-    act = _expert_act(activation, "experts_apply")
-    _check(lib().vk_experts_gate_up(_p(x), W, _p(w_gate_up), ff, top, _p(ids), E, act, ctypes.c_float(limit), ctypes.c_float(alpha), _p(act_buf), T,
+    act = _expert_act(activation, "experts_apply", gated)
+    _check(lib().vk_experts_gate_up(_p(x), W, _p(w_gate_up), ff, top, _p(ids), E, int(gated), act, ctypes.c_float(limit), ctypes.c_float(alpha), _p(act_buf), T,
                                     _dt(x), _stream()), "experts_gate_up")
     _check(lib().vk_experts_down(_p(act_buf), ff, _p(w_down), W, top, _p(ids), _p(wts), _p(y), E, _p(x), T, _dt(x), _stream()), "experts_down")
     return y
@@ -1450,7 +1473,7 @@ def experts_grouped_rows(tokens: int, top: int, E: int) -> int:
 
 def experts_grouped_takes(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor) -> bool:
     """Whether the tensor-core form takes these operands: bfloat16, 16-byte aligned, sizes that are multiples of 8."""
-    ff, W = w_gate_up.shape[1] // 2, x.shape[1]
+    ff, W = w_down.shape[2], x.shape[1]
     return (x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and w_down.dtype == torch.bfloat16 and W % 8 == 0 and ff % 8 == 0
             and x.stride(0) == W and x.data_ptr() % 16 == 0 and w_gate_up.data_ptr() % 16 == 0 and w_down.data_ptr() % 16 == 0)
 
@@ -1458,36 +1481,38 @@ def experts_grouped_takes(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torc
 def experts_apply_grouped(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, pos: torch.Tensor,
                           row_token: torch.Tensor, tile_group: torch.Tensor, xs: torch.Tensor, act_buf: torch.Tensor, o: torch.Tensor,
                           y: torch.Tensor, activation: str = "silu", limit: float = 0.0, alpha: float = 1.702,
-                          gu_buf: Optional[torch.Tensor] = None) -> torch.Tensor:
+                          gu_buf: Optional[torch.Tensor] = None, gated: bool = True) -> torch.Tensor:
     """experts_apply on the tensor cores: the tokens' copies are put expert by expert into xs [rows, W] (rows =
     experts_grouped_rows(T, top, E); pos [T, top], row_token [rows], tile_group [rows / 128] int32), two products of row groups give
     act_buf [rows, ff] (bfloat16) and o [rows, W] (float32), and y [T, W] (float32) += the weighted rows of each token.
-    activation "clamped" (with gu_buf [rows, 2 ff] bfloat16): the first product leaves gate and up, and glu_clamped follows."""
+    activation "clamped" (with gu_buf [rows, 2 ff] bfloat16): the first product leaves gate and up, and glu_clamped follows.  gated False: as in
+    experts_apply."""
     _req(x, "x", torch.bfloat16, 2); _req(y, "y", torch.float32, 2); _req(o, "o", torch.float32, 2); _req(xs, "xs", torch.bfloat16, 2)
     _req(act_buf, "act_buf", torch.bfloat16, 2); _req(pos, "pos", torch.int32, 2); _req(row_token, "row_token", torch.int32, 1)
     _req(tile_group, "tile_group", torch.int32, 1)
     T, W = x.shape
-    E, two_ff, _ = w_gate_up.shape
-    ff, top = two_ff // 2, ids.shape[1]
+    E, per = w_gate_up.shape[0], 2 if gated else 1
+    ff, top = w_gate_up.shape[1] // per, ids.shape[1]
     rows = experts_grouped_rows(T, top, E)
-    if (not experts_grouped_takes(x, w_gate_up, w_down) or w_gate_up.shape != (E, 2 * ff, W) or w_down.shape != (E, W, ff) or y.shape != (T, W)
+    if (not experts_grouped_takes(x, w_gate_up, w_down) or w_gate_up.shape != (E, per * ff, W) or w_down.shape != (E, W, ff) or y.shape != (T, W)
             or xs.shape != (rows, W) or act_buf.shape != (rows, ff) or o.shape != (rows, W) or pos.shape != (T, top) or row_token.shape != (rows,)
             or tile_group.shape != (rows // 128,)):
         raise KernelError("experts_apply_grouped: shapes do not fit")
-    act = _expert_act(activation, "experts_apply_grouped")
-    act = 0 if activation == "silu" else act
-    if act == 4:
+    act = _expert_act(activation, "experts_apply_grouped", gated)
+    act = 0 if gated and activation == "silu" else act
+    clamped = gated and act == 4
+    if clamped:
         if gu_buf is None or gu_buf.shape != (rows, 2 * ff):
             raise KernelError("experts_apply_grouped: the clamped form needs gu_buf [rows, 2 ff]")
         _req(gu_buf, "gu_buf", torch.bfloat16, 2)
     _check(lib().vk_experts_sort(_p(ids), T, top, E, rows, _p(pos), _p(row_token), _p(tile_group), _stream()), "experts_sort")
     _check(lib().vk_experts_gather(_p(x), W, _p(row_token), _p(xs), rows, _dt(x), _stream()), "experts_gather")
-    if act == 4:
+    if clamped:
         _check(lib().vk_linear_tcgen05_grouped(_p(xs), _p(w_gate_up), _p(gu_buf), rows, 2 * ff, W, W, E, _p(tile_group), 0, 0, 0, _p(error_word()),
                                                _stream()), "linear_tcgen05_grouped")
         glu_clamped(gu_buf, act_buf, limit, alpha)
     else:
-        _check(lib().vk_linear_tcgen05_grouped(_p(xs), _p(w_gate_up), _p(act_buf), rows, ff, W, W, E, _p(tile_group), 0, 1, act, _p(error_word()),
+        _check(lib().vk_linear_tcgen05_grouped(_p(xs), _p(w_gate_up), _p(act_buf), rows, ff, W, W, E, _p(tile_group), 0, int(gated), act, _p(error_word()),
                                                _stream()), "linear_tcgen05_grouped")
     _check(lib().vk_linear_tcgen05_grouped(_p(act_buf), _p(w_down), _p(o), rows, W, ff, ff, E, _p(tile_group), 1, 0, 0, _p(error_word()),
                                            _stream()), "linear_tcgen05_grouped")
@@ -1585,14 +1610,18 @@ def gla(proj: torch.Tensor, a_off: int, a2t: torch.Tensor, bias: torch.Tensor, t
 def mixed_attn_prepare(proj: torch.Tensor, positions: torch.Tensor, slot_mapping: Optional[torch.Tensor], q_norm: Optional[torch.Tensor],
                        k_norm: Optional[torch.Tensor], eps: float, freq: Optional[torch.Tensor], dims: int, vfreq: Optional[torch.Tensor],
                        q_out: torch.Tensor, cache_layer: Optional[torch.Tensor], nh: int, nkv: int, hd: int, vd: int, page_size: int,
-                       bias: Optional[torch.Tensor] = None, v_mult: float = 1.0, off: int = 0) -> torch.Tensor:
+                       bias: Optional[torch.Tensor] = None, v_mult: float = 1.0, off: int = 0, neighbours: bool = False,
+                       v_from_k: bool = False) -> torch.Tensor:
     """From the columns [q | k | v] at `off` of the first product's float32 rows, plus `bias` [its columns] if given: q and k heads / rms * weight (eps < 0: no norm),
     v times v_mult, the first `dims` values of q and k turned
-    in pairs (i, i + dims / 2) by position * freq[i]; v turned over all its pairs by position * vfreq[m] (None: not); q to q_out, k and v
-    into the layer's pages at slot_mapping (-1: no write)."""
+    in pairs (i, i + dims / 2), or (2i, 2i + 1) with neighbours, by position * freq[i]; v turned over all its pairs by position * vfreq[m] (None: not); q to q_out, k and v
+    into the layer's pages at slot_mapping (-1: no write).  v_from_k: the columns are [q | k], and v is k before norm and rotation."""
     _req(proj, "proj", torch.float32, 2); _req(positions, "positions", torch.int32, 1); _req(q_out, "q_out", dims=2)
     T, N = proj.shape
-    if off < 0 or N < off + (nh + nkv) * hd + nkv * vd or q_out.shape != (T, nh * hd) or positions.shape[0] < T:
+    cols = (nh + nkv) * hd + (0 if v_from_k else nkv * vd)
+    if v_from_k and (vd != hd or vfreq is not None):
+        raise KernelError("mixed_attn_prepare: values that are the projected keys have their size and are not turned")
+    if off < 0 or N < off + cols or q_out.shape != (T, nh * hd) or positions.shape[0] < T:
         raise KernelError("mixed_attn_prepare: shapes do not fit the head counts")
     for v, n, name in ((q_norm, hd, "q_norm"), (k_norm, hd, "k_norm"), (freq, dims // 2, "freq"), (vfreq, vd // 2, "vfreq")):
         if v is not None:
@@ -1603,7 +1632,7 @@ def mixed_attn_prepare(proj: torch.Tensor, positions: torch.Tensor, slot_mapping
         raise KernelError("mixed_attn_prepare: a rotation needs its frequencies")
     if bias is not None:
         _req(bias, "bias", torch.float32, 1)
-        if bias.shape[0] != (nh + nkv) * hd + nkv * vd:
+        if bias.shape[0] != cols:
             raise KernelError("mixed_attn_prepare: the bias does not fit the head counts")
     if cache_layer is not None:
         _req(cache_layer, "cache_layer", q_out.dtype); _req(slot_mapping, "slot_mapping", torch.int32, 1)
@@ -1611,7 +1640,8 @@ def mixed_attn_prepare(proj: torch.Tensor, positions: torch.Tensor, slot_mapping
             raise KernelError("mixed_attn_prepare: the cache layer does not fit the page size")
     _check(lib().vk_mixed_attn_prepare(ctypes.c_void_p(proj.data_ptr() + 4 * off), N, _p(positions), _p(slot_mapping if cache_layer is not None else None), _p(q_norm), _p(k_norm),
                                        ctypes.c_float(eps), _p(freq if dims else None), dims, _p(vfreq), _p(q_out), _p(cache_layer), T, nh, nkv, hd, vd,
-                                       page_size, _p(bias), ctypes.c_float(v_mult), _dt(q_out), _stream()), "mixed_attn_prepare")
+                                       page_size, _p(bias), ctypes.c_float(v_mult), int(bool(neighbours)), int(bool(v_from_k)), _dt(q_out), _stream()),
+           "mixed_attn_prepare")
     return q_out
 
 
@@ -1823,4 +1853,93 @@ def ssd(proj: torch.Tensor, off: int, conv_w: torch.Tensor, conv_b: Optional[tor
                                        N, P, _dt(out), _stream()), "ssd_recurrence")
     _check(L.vk_ssd_gate(_p(y), _p(proj), width, z_off, x_off, _p(norm_w), ctypes.c_float(eps), ctypes.c_float(mult), parts, _p(out), out_ld,
                          _p(ctx.seg_starts), _p(ctx.seg_slots), ctx.num_segments, _p(state), stride, T, H, G, N, P, taps, _dt(out), _stream()), "ssd_gate")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# Sublayers whose results are scaled value by value; a per-layer input from the token itself
+# ---------------------------------------------------------------------------
+
+TOKEN_SIDE_MAX_ROWS = 32        # beyond this many tokens the per-layer input's two products run as products
+
+
+def _step_args(x, y, scale, table, ids, add, norm, out, name):
+    _req(x, "x", torch.float32, 2)
+    T, n = x.shape
+    if y is not None:
+        _req(y, "y", torch.float32, 2)
+        if y.shape != x.shape:
+            raise KernelError(f"{name}: y is not x's shape")
+    if scale is not None and y is None:
+        raise KernelError(f"{name}: a scale without the rows it scales")
+    for v, what in ((scale, "scale"), (add, "add"), (None if norm is None else norm[0], "norm weight"), (None if norm is None else norm[1], "norm bias")):
+        if v is not None:
+            _req(v, what, torch.float32, 1)
+            if v.shape[0] != n:
+                raise KernelError(f"{name}: {what} does not fit the width")
+    if out is not None:
+        _req(out, "out", dims=2)
+        if out.shape != x.shape:
+            raise KernelError(f"{name}: out is not x's shape")
+    elif norm is not None:
+        raise KernelError(f"{name}: a norm needs somewhere to go")
+    if table is not None:
+        _req(table, "table", out.dtype if out is not None else None, 2)
+        if table.shape[1] != n or ids is None:
+            raise KernelError(f"{name}: the table's rows are not of the width")
+    if ids is not None:
+        _req(ids, "ids", torch.int32, 1)
+        if ids.shape[0] < T:
+            raise KernelError(f"{name}: fewer ids than rows")
+    kind = out if out is not None else table
+    wn, bn = norm if norm is not None else (None, None)
+    return T, n, wn, bn, 0 if kind is None else _dt(kind)
+
+
+def residual_step(x: torch.Tensor, y: Optional[torch.Tensor] = None, scale: Optional[torch.Tensor] = None, *, z: Optional[torch.Tensor] = None,
+                  z_norm: Optional[torch.Tensor] = None, mult: float = 1.0, table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
+                  add: Optional[torch.Tensor] = None, norm: Optional[tuple] = None, out: Optional[torch.Tensor] = None, eps: float = 0.0) -> Optional[torch.Tensor]:
+    """x (float32 [T, n]) += scale . y, then y = 0;  x += mult * z / sqrt(mean(z^2) + eps) . z_norm;  x += table[ids];  x += add;  out = the layer norm of
+    x with norm = (weight, bias), or without norm x itself, in out's dtype.  What is not given is left out (y without scale is only zeroed)."""
+    T, n, wn, bn, dt = _step_args(x, y, scale, table, ids, add, norm, out, "residual_step")
+    if z is not None:
+        _req(z, "z", torch.float32, 2); _req(z_norm, "z_norm", torch.float32, 1)
+        if z.shape != x.shape or z_norm.shape[0] != n:
+            raise KernelError("residual_step: z does not fit x")
+    _check(lib().vk_residual_step(_p(x), _p(y), _p(scale), _p(z), _p(z_norm if z is not None else None), _p(table), _p(ids if table is not None else None),
+                                  0 if table is None else table.shape[0], _p(add), _p(wn), _p(bn), _p(out), T, n, ctypes.c_float(eps), ctypes.c_float(mult),
+                                  dt, _stream()), "residual_step")
+    return out
+
+
+def token_gate(a: torch.Tensor, side: torch.Tensor, off: int, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out [T, dim] = gelu_tanh(a) * side[ids, off : off + dim]; a float32 [T, dim], side [vocab, *] in out's dtype."""
+    _req(a, "a", torch.float32, 2); _req(out, "out", dims=2); _req(side, "side", out.dtype, 2); _req(ids, "ids", torch.int32, 1)
+    T, dim = a.shape
+    if out.shape != a.shape or ids.shape[0] < T or off < 0 or off + dim > side.shape[1]:
+        raise KernelError("token_gate: shapes do not fit")
+    _check(lib().vk_token_gate(_p(a), _p(side), side.shape[1], off, _p(ids), side.shape[0], _p(out), T, dim, _dt(out), _stream()), "token_gate")
+    return out
+
+
+def token_side_takes(dtype: torch.dtype, rows: int, n: int, dim: int) -> bool:
+    """Whether residual_step and the per-layer input run as one kernel: few tokens (not in the exact 32-bit routing), a row that fits."""
+    fn = lib().vk_token_side_smem
+    fn.restype = ctypes.c_size_t
+    return rows <= TOKEN_SIDE_MAX_ROWS and not (dtype == torch.float32 and _float32_exact) and int(fn(n, dim)) <= 200 * 1024
+
+
+def token_side(x: torch.Tensor, y: Optional[torch.Tensor], scale: Optional[torch.Tensor], gate: torch.Tensor, proj: torch.Tensor, side: torch.Tensor, off: int,
+               z_norm: torch.Tensor, ids: torch.Tensor, *, mult: float = 1.0, table: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None,
+               norm: Optional[tuple] = None, out: Optional[torch.Tensor] = None, eps: float = 0.0) -> Optional[torch.Tensor]:
+    """residual_step with z = proj g, g = gelu_tanh(gate (x + scale . y)) * side[ids, off : off + dim], in one launch (gate [dim, n], proj [n, dim] and
+    side [vocab, *] in one dtype, which is out's and the table's)."""
+    T, n, wn, bn, _ = _step_args(x, y, scale, table, ids, add, norm, out, "token_side")
+    _req(gate, "gate", dims=2); _req(proj, "proj", gate.dtype, 2); _req(side, "side", gate.dtype, 2); _req(z_norm, "z_norm", torch.float32, 1)
+    dim = gate.shape[0]
+    if (gate.shape[1] != n or proj.shape != (n, dim) or off < 0 or off + dim > side.shape[1] or z_norm.shape[0] != n
+            or any(t is not None and t.dtype != gate.dtype for t in (out, table)) or (table is not None and table.shape[0] != side.shape[0])):
+        raise KernelError("token_side: shapes or dtypes do not fit")
+    _check(lib().vk_token_side(_p(x), _p(y), _p(scale), _p(gate), _p(proj), dim, _p(side), side.shape[1], off, _p(z_norm), _p(table), _p(ids), side.shape[0],
+                               _p(add), _p(wn), _p(bn), _p(out), T, n, ctypes.c_float(eps), ctypes.c_float(mult), _dt(gate), _stream()), "token_side")
     return out

@@ -16,7 +16,10 @@ gate is one of the gated epilogues' activations, or "clamped": the clamped gated
 
 The scored router (`scored`, a ScoredRouter): scores s = softmax(W_router xn) over ALL experts; the choice goes by s + correction, inside the best
 groups of neighbouring experts; weights s / (sum of the chosen s + 1e-20) * scale.  The last rows of its matrix may be identities, "experts"
-without weights whose output is xn itself."""
+without weights whose output is xn itself.  Or the scores are s = sigmoid(W_router xn), each for itself, and the weights s * scale as they are.
+
+An expert is gated, as above, or (gated=False) W_down act(W_up xn), act one of ops.DENSE_ACTIVATIONS.  Where the weight multiplies an expert's INPUT
+(weigh_input) and act is homogeneous of degree d, act(w z) = w^d act(z), the output is multiplied by w^d instead: no other kernel, no rounding of w xn."""
 from __future__ import annotations
 
 import math
@@ -125,6 +128,7 @@ class ScoredRouter:
     keep: int = 1
     identities: int = 0
     scale: float = 1.0
+    sigmoid: bool = False
 
 
 class RoutedExperts(FeedForward):
@@ -139,11 +143,12 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, hidden: int, intermediate: int, experts: int, top: int, w_router: Optional[torch.Tensor], b_router: Optional[torch.Tensor],
                  w_gate_up: torch.Tensor, w_down: torch.Tensor, shared: Optional[FeedForward] = None, activation: str = "silu",
-                 table: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 1.702, scored: Optional[ScoredRouter] = None):
-        """With `scored` w_router is [E + identities, hidden] and there is no b_router.  Either w_router (float32 [E, hidden], with or without b_router) or table (int32 [vocab, >= top]: the experts of every token
+                 table: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 1.702, scored: Optional[ScoredRouter] = None,
+                 gated: bool = True, weigh_input: bool = False):
+        """gated False: w_gate_up is W_up, [E, intermediate, hidden].  weigh_input: the router's weights multiply the experts' inputs.  With `scored` w_router is [E + identities, hidden] and there is no b_router.  Either w_router (float32 [E, hidden], with or without b_router) or table (int32 [vocab, >= top]: the experts of every token
         id, each weighted 1 / top).  activation: one of the gated epilogues' or "clamped" (with limit and alpha)."""
         E = experts
-        if w_gate_up.shape != (E, 2 * intermediate, hidden) or w_down.shape != (E, hidden, intermediate):
+        if w_gate_up.shape != (E, (2 if gated else 1) * intermediate, hidden) or w_down.shape != (E, hidden, intermediate):
             raise ValueError("the experts' weights do not fit the sizes")
         if (w_router is None) == (table is None):
             raise ValueError("the experts are chosen by a router or by a table, one of the two")
@@ -166,7 +171,11 @@ class RoutedExperts(FeedForward):
         if activation == "clamped" and not limit > 0:
             raise ValueError("the clamp's limit is positive")
         self.hidden, self.intermediate, self.E, self.top, self.activation, self.shared = hidden, intermediate, E, int(top), activation, shared
-        self.limit, self.alpha, self.scored = float(limit), float(alpha), scored
+        if not gated and activation not in ops.DENSE_ACTIVATIONS:
+            raise ValueError(f"activation {activation!r} is not one of {sorted(ops.DENSE_ACTIVATIONS)}")
+        if weigh_input and (gated or activation != "relu2" or scored is None or not scored.sigmoid or scored.identities or scored.scale < 0):
+            raise ValueError("weights on the experts' inputs: ungated experts with relu squared, and a router whose weights are not negative")
+        self.limit, self.alpha, self.scored, self.gated, self.weigh_input = float(limit), float(alpha), scored, bool(gated), bool(weigh_input)
         self.correction = None if scored is None or scored.correction is None else scored.correction.to(torch.float32).contiguous()
         self.w_router = None if w_router is None else w_router.to(torch.float32).contiguous()
         self.b_router = None if b_router is None else b_router.to(torch.float32).contiguous()
@@ -190,7 +199,8 @@ class RoutedExperts(FeedForward):
         if self.table is not None:
             ops.experts_route_table(ctx.tokens, self.table, self.E, self.top, ids, wts)
         elif self.scored is not None:
-            ops.experts_route_scored(xn, self.w_router, self.correction, self.top, self.scored.groups, self.scored.keep, self.scored.scale, ids, wts)
+            ops.experts_route_scored(xn, self.w_router, self.correction, self.top, self.scored.groups, self.scored.keep, self.scored.scale, ids, wts,
+                                     self.scored.sigmoid, self.weigh_input)
         else:
             ops.experts_route(xn, self.w_router, self.b_router, self.top, ids, wts)
         if T * self.top >= self.GROUPED_FROM and ops.experts_grouped_takes(xn, self.w_gate_up, self.w_down):
@@ -205,10 +215,11 @@ class RoutedExperts(FeedForward):
                                       ws.flat(f"moe.tile_group/{key}", rows_max // 128, torch.int32)[:rows // 128], xs, act, o, residual, self.activation,
                                       self.limit, self.alpha,
                                       None if self.activation != "clamped" else
-                                      ws.flat(f"moe.gu/{key}/{self.intermediate}", rows_max * 2 * self.intermediate, ctx.dtype)[:rows * 2 * self.intermediate].view(rows, 2 * self.intermediate))
+                                      ws.flat(f"moe.gu/{key}/{self.intermediate}", rows_max * 2 * self.intermediate, ctx.dtype)[:rows * 2 * self.intermediate].view(rows, 2 * self.intermediate),
+                                      gated=self.gated)
         else:
             act = ws.flat(f"moe.act/{self.top}/{self.intermediate}", ws.max_tokens * self.top * self.intermediate, ctx.dtype)
             ops.experts_apply(xn, self.w_gate_up, self.w_down, ids, wts, act[:T * self.top * self.intermediate].view(T * self.top, self.intermediate),
-                              residual, self.activation, self.limit, self.alpha)
+                              residual, self.activation, self.limit, self.alpha, self.gated)
         if self.shared is not None:
             self.shared.forward(xn, ctx, residual)

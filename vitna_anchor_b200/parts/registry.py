@@ -32,7 +32,7 @@ def make_part(kind: str, name: str, **params):
 
 def _register_builtin() -> None:
     from .attention import PagedAttention
-    from .block import OutputNormBlock, PreNormBlock, SandwichNormBlock
+    from .block import OutputNormBlock, PreNormBlock, SandwichNormBlock, ScaledResidualBlock
     from .gla import GatedLinearAttention
     from .mixed_attention import MixedHeadAttention
     from .parallel import ParallelMixer
@@ -69,6 +69,7 @@ def _register_builtin() -> None:
     register_part("block", "pre_norm", PreNormBlock)
     register_part("block", "output_norm", OutputNormBlock)
     register_part("block", "sandwich_norm", SandwichNormBlock)
+    register_part("block", "scaled_residual", ScaledResidualBlock)
     register_part("block", "hyper", HyperBlock)
 
 

@@ -37,6 +37,23 @@ class NoPositionEncoding(PositionEncoding):
     """Nothing is added or rotated."""
 
 
+def banded_frequencies(base: float, dims: int, scaling=None):
+    """Frequencies of a rotation over `dims` values, f_i = base^(-2i/dims), i < dims/2, rescaled by wavelength.
+
+    With scaling = (factor, low, high, original) and l = 2 pi / f: f stays where l < original / high, becomes f / factor where l > original / low,
+    and between the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low) (the Llama 3.1 recipe).  Worked out in float64
+    on the host; -> float32 [dims/2] array."""
+    if dims % 2:
+        raise ValueError("a rotation turns an even number of values")
+    f = np.power(float(base), -2.0 * np.arange(dims // 2, dtype=np.float64) / max(dims, 1))
+    if scaling is not None:
+        factor, low, high, original = (float(v) for v in scaling)
+        length = 2.0 * np.pi / f
+        s = (original / length - low) / (high - low) if high != low else np.ones_like(f)
+        f = np.where(length < original / high, f, np.where(length > original / low, f / factor, (1.0 - s) * f / factor + s * f))
+    return f.astype(np.float32)
+
+
 def blended_frequencies(base: float, dims: int, scaling=None):
     """Frequencies of a rotation over `dims` values, f_i = base^(-2i/dims), i < dims/2, and the factor on cos and sin.
 
