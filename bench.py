@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, as one JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
-                    [--model 135M|360M|1.7B] [--workload decode|mixed|prefill8k|lupanex|siparax|manatar|tinevik|lirutar]
+                    [--model 135M|360M|1.7B] [--workload decode|mixed|prefill8k|lupanex|siparax|manatar|tinevik|lirutar|zolapel]
 
 The default run is SmolLM2-135M's sizes with random weights (N(0, 0.02), norm weights 1, seed 0) in
 bfloat16, a batch of 8 requests each decoding from its own 2,048-token random prompt, cache context
@@ -33,6 +33,9 @@ token uses: the same measurements (TINEVIK_SIZES below).
 --workload lirutar: the Lirutar design (attention over a window and a state-space mixer side by side in every layer, looped layers,
 experts chosen by corrected scores inside groups) beside Tinevik at equal width, runs of a layer, heads and feed-forward weights a token
 uses: the same measurements (LIRUTAR_SIZES below).
+--workload zolapel: the Zolapel design (attention over a window whose values are the projected keys, ungated experts weighed on their inputs,
+scaled sublayers, a per-layer input from the token, looped layers) beside Lirutar at equal width, runs of a layer, attention work and
+feed-forward weights a token uses: the same measurements (ZOLAPEL_SIZES below).
 --workload prefill8k: one 8,192-token prompt, in one step and in portions of 2,048 through the scheduler.
 
 --impl reference builds nothing of this repository's engine: it runs the unmodified reference program
@@ -548,7 +551,7 @@ def kind_of(launch):
         return "ssd"
     if launch == "latent_expand_gate":
         return "expand"
-    if launch in ("sandwich_step", "xielu", "mixed_attn_prepare", "embed_scaled", "pass_input"):
+    if launch in ("sandwich_step", "xielu", "mixed_attn_prepare", "embed_scaled", "pass_input", "residual_step", "token_gate", "token_side", "embed_rows"):
         return "between"
     if launch in ("embed_hashed", "residual_norm_step", "glu_clamped", "diff_attn_prepare", "diff_attn_combine"):
         return "between"
@@ -935,6 +938,71 @@ def lirutar_run(a, pk, clocks):
     return results
 
 
+# ---------------------------------------------------------------------------------------------------------------
+# --workload zolapel
+# ---------------------------------------------------------------------------------------------------------------
+
+# Zolapel beside Lirutar, the engine's closest design: layer norms, a windowed rotary attention with grouped heads, routed experts on the same
+# grouped products, layers that run twice.  Equal width, runs of a layer (six layers of which two run twice: eight), heads, window, key and value
+# values together (at width 1,024 Lirutar's heads have 64 and 128, Zolapel's 96 and 96), and weights a token uses in the feed-forwards (4 of 16
+# ungated experts of 3/8 the width against 2 of 8 gated ones of a quarter and a shared one of half; Lirutar's first layer is dense).  Lirutar's layers
+# have a state-space mixer beside the attention, Zolapel's an input from the token.
+ZOLAPEL_SIZES = {
+    "w1024": dict(LIRUTAR_SIZES["w1024"], dim=96, side=128),
+    "w2048": dict(LIRUTAR_SIZES["w2048"], side=256),
+}
+ZOLAPEL_EXPERTS, ZOLAPEL_TOP = 16, 4
+
+
+def zolapel_config(sz):
+    rot = dict(base=500000.0, dims=sz["dim"], scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))
+    mixer = dict(heads=2 * sz["heads"], kv_heads=sz["kv"], dim=sz["dim"], vdim=sz["dim"], scale=sz["dim"] ** -0.5, rot=rot, mask=dict(size=sz["window"]))
+    mlp = dict(kind="moe", expert=dict(ff=3 * sz["ff"] // 8), router=dict(experts=ZOLAPEL_EXPERTS, top=ZOLAPEL_TOP))
+    n = sz["layers"] - (LIRUTAR_LOOP["stop"] - LIRUTAR_LOOP["start"]) * (LIRUTAR_LOOP["times"] - 1)
+    return dict(architecture="Zolapel", vocab=LUPANEX_VOCAB, width=sz["width"], norm=dict(eps=1e-6), residual_mult=0.8, token_side=dict(dim=sz["side"]),
+                loop=LIRUTAR_LOOP, layers=[dict(type="attention", mixer=mixer, mlp=mlp) for _ in range(n)])
+
+
+def zolapel_work(sz, T):
+    """Algorithmic work of one T-token prompt, by kind of kernel: (flops, bytes)."""
+    W, L, H, G, d, win, side = sz["width"], sz["layers"], 2 * sz["heads"], sz["kv"], sz["dim"], sz["window"], sz["side"]
+    rows = H * d + G * d + H
+    seen = float(T) * (T + 1) / 2 if win >= T else float(T) * win - win * (win - 1) / 2.0        # (query, key) pairs inside the window
+    e_ff = 3 * sz["ff"] // 8
+    return {
+        "product": (2.0 * T * L * W * (rows + H * d + 2 * side), 0.0),
+        "attention": (L * 2.0 * seen * H * 2 * d, 0.0),
+        "experts": (L * 2.0 * T * ZOLAPEL_TOP * 2 * W * e_ff, L * ZOLAPEL_EXPERTS * 2.0 * W * e_ff * 2),
+        "between": (0.0, L * T * (W * (18.0 + 18.0 + 14.0) + 4.0 * rows + 2.0 * (H + 2 * G) * d + 8.0 * side) + T * W * 8.0),
+    }
+
+
+def zolapel_run(a, pk, clocks):
+    import torch
+    from vitna_anchor_b200.engine.loading import random_model_on_device
+    results = {}
+    for name, sz in ZOLAPEL_SIZES.items():
+        row = {}
+        for which, cfg, work in (("zolapel", zolapel_config(sz), zolapel_work(sz, PREFILL_TOKENS)),
+                                 ("lirutar", lirutar_config(LIRUTAR_SIZES[name]), lirutar_work(LIRUTAR_SIZES[name], PREFILL_TOKENS))):
+            model = random_model_on_device(cfg, 0)
+            if model.max_positions > CONTEXT:
+                model.max_positions = CONTEXT           # the design has no limit of its own; the run's cache has
+            pf = prefill_run(model, None, clocks, repeats=3)
+            dec = decode_run(model, a.batch, min(a.steps, 32), a.warmup, clocks, with_e2e=False)
+            flops = sum(f for f, _ in work.values())
+            row[which] = {"weights_mb": round(model.step_weight_bytes() / 1e6, 1),
+                          "prefill_2048": {"tokens_per_s": round(pf["value"]), "ms": round(pf["ms"], 3),
+                                           "frac_bf16": round(flops / (pf["ms"] * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)},
+                          f"decode_b{a.batch}": {"tokens_per_s": round(dec["value"]), "ms_per_step": round(dec["ms_per_step"], 4),
+                                                 "frac_hbm": round(dec["gbs"] / pk["hbm_gbs"], 4), "launches_per_step": dec["launches"] // min(a.steps, 32)},
+                          "prompt_by_kind": prompt_by_kind(model, work, pk)}
+            del model
+            torch.cuda.empty_cache()
+        results[name] = row
+    return results
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -943,10 +1011,11 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--model", default="135M", choices=sorted(MODELS), help="layer sizes: SmolLM2-135M (the default), 360M or 1.7B")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "prefill8k", "lupanex", "siparax", "manatar", "tinevik", "lirutar"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "prefill8k", "lupanex", "siparax", "manatar", "tinevik", "lirutar",
+                                                              "zolapel"],
                     help="decode (the default line), mixed (32 requests, 512-token portions beside decodes), prefill8k, lupanex "
                          "(the Lupanex design beside a Llama model of equal size), siparax and manatar (those designs beside Lupanex), "
-                         "tinevik (that design beside Manatar with routed feed-forwards), lirutar (that design beside Tinevik)")
+                         "tinevik (that design beside Manatar with routed feed-forwards), lirutar (that design beside Tinevik), zolapel (that design beside Lirutar)")
     ap.add_argument("--no-points", action="store_true", help="skip the other batches, models and the prefill")
     ap.add_argument("--only-prefill", action="store_true", help="run the prefill measurement alone (for profiling)")
     ap.add_argument("--profile-region", default="", choices=["", "decode", "prefill"],
@@ -1014,6 +1083,15 @@ def main():
         r = lirutar_run(a, pk, clocks)
         clocks.stop()
         print(json.dumps({"metric": "Lirutar beside Tinevik at equal width, runs of a layer, heads and feed-forward weights a token uses: tokens/s "
+                          f"of a 2,048-token prompt and of batch-{a.batch} decoding from 2,048-token prompts; a prompt's time by kind of kernel "
+                          "against its roofline", "impl": "ours", "dtype": "bf16",
+                          "data": "synthetic: random weights drawn on the device, uniform-random token ids", "peaks": pk, "sizes": r,
+                          "clocks": clocks.summary()}))
+        return 0
+    if a.workload == "zolapel":
+        r = zolapel_run(a, pk, clocks)
+        clocks.stop()
+        print(json.dumps({"metric": "Zolapel beside Lirutar at equal width, runs of a layer, attention work and feed-forward weights a token uses: tokens/s "
                           f"of a 2,048-token prompt and of batch-{a.batch} decoding from 2,048-token prompts; a prompt's time by kind of kernel "
                           "against its roofline", "impl": "ours", "dtype": "bf16",
                           "data": "synthetic: random weights drawn on the device, uniform-random token ids", "peaks": pk, "sizes": r,

@@ -213,8 +213,8 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
     auto places = [&](int j, int& a, int& b) {
         if (!neighbours && j < half) { a = j; b = j + half; } else { a = 2 * j; b = a + 1; }
     };
-    float2 v[P];
-    auto fetch = [&](int h) {
+    float2 v[P], ahead[2][P];                           // this head's row, and the warp's next two
+    auto fetch = [&](int h, float2* v) {
         const float* row = in + (size_t)h * hd;
 #pragma unroll
         for (int p = 0; p < P; p++) {
@@ -225,15 +225,17 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
             v[p] = b == a + 1 ? *reinterpret_cast<const float2*>(row + a) : make_float2(row[a], row[b]);
         }
     };
-    if (warp < n_qk) fetch(warp);
+    fetch(min(warp, n_qk - 1), v);
+    if (warp + nwarps < n_qk) fetch(warp + nwarps, ahead[0]);
+    if (warp + 2 * nwarps < n_qk) fetch(warp + 2 * nwarps, ahead[1]);
     const float pos = (float)positions[t];
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         const float ang = pos * freq[i];
-        nr_turn[2 * i] = cosf(ang);
-        nr_turn[2 * i + 1] = sinf(ang);
+        sincosf(ang, &nr_turn[2 * i + 1], &nr_turn[2 * i]);
     }
     __syncthreads();
-    for (int h = warp; h < n_heads; h += nwarps) {
+    int round = 0;
+    for (int h = warp; h < n_heads; h += nwarps, round++) {
         if (h >= n_qk) {                                // a value head of its own
             if (s < 0) continue;
             const int g = h - n_qk;
@@ -242,7 +244,12 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
             for (int d = lane; d < vd; d += 32) dst[d] = from_f32<T>(row[d] * v_mult);
             continue;
         }
-        if (h != warp) fetch(h);
+        if (round == 1 || round == 2) {
+#pragma unroll
+            for (int p = 0; p < P; p++) v[p] = round == 1 ? ahead[0][p] : ahead[1][p];
+        } else if (round > 2) {
+            fetch(h, v);
+        }
         const bool key = h >= nh;
         if (key && s < 0) continue;
         const float* w = key ? kn_w : qn_w;

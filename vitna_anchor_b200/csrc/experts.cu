@@ -15,6 +15,12 @@
 //  experts_down      y[token] += sum_k weight_k W_down,e_k act[token, k], the experts of a token summed in the order of its list, so
 //                    that the sum does not depend on what else is in the batch.
 //
+//  experts_shared_up, experts_shared_down   the same two for a few tokens that share experts: a block an expert and some columns, which reads its rows
+//                    of the weights once for all of the step's (token, k) pairs that chose the expert (in passes of up to four pairs whose
+//                    input rows lie in shared memory); the second leaves a float32 row a pair (or, where a token has one expert, adds it
+//                    to y) and experts_combine adds them up.  The sums run in the order of the two kernels above, so that the
+//                    result is the same bits.
+//
 // For a prompt's portion in bfloat16 the experts' products run on the tensor cores as products of row groups (linear_tcgen05.cu):
 //  experts_sort      one block: counts the copies a group (an expert) gets, gives every group whole tiles of 128 rows one after another,
 //                    and writes for each (token, k) its row, for each row its token (-1: a fill row), for each tile its group
@@ -306,6 +312,112 @@ __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__
     }
 }
 
+constexpr int ES_PAIRS = 4, ES_STREAMS = 4, ES_MAX_PAIRS = 256;        // pairs a pass; weight rows a warp reads side by side; pairs a step
+enum { ES_UP = 0, ES_GATED = 1, ES_DOWN = 2 };
+
+template <typename T, int NP>
+__device__ __forceinline__ void es_dots(const T* const* w, const T* rows, int n, int lane, float (*acc)[ES_STREAMS]) {
+    constexpr int V = Vec16<T>::N;
+#pragma unroll
+    for (int p = 0; p < NP; p++)
+#pragma unroll
+        for (int s = 0; s < ES_STREAMS; s++) acc[p][s] = 0.0f;
+#pragma unroll 2
+    for (int i = lane * V; i < n; i += 32 * V) {
+        float f[ES_STREAMS][V];
+#pragma unroll
+        for (int s = 0; s < ES_STREAMS; s++) load16<T>(w[s] + i, f[s]);
+#pragma unroll
+        for (int p = 0; p < NP; p++) {
+            float v[V];
+            load16<T>(rows + (size_t)p * n + i, v);
+#pragma unroll
+            for (int s = 0; s < ES_STREAMS; s++)
+#pragma unroll
+                for (int e = 0; e < V; e++) acc[p][s] = fmaf(v[e], f[s][e], acc[p][s]);
+        }
+    }
+#pragma unroll
+    for (int p = 0; p < NP; p++)
+#pragma unroll
+        for (int s = 0; s < ES_STREAMS; s++) acc[p][s] = warp_sum(acc[p][s]);
+}
+
+// grid (E, column groups).  n: the length of a row of the weights and of the inputs; cols: output columns.  ES_GATED, ES_UP: in is x [tokens][n], out
+// [pairs][cols] in T; ES_DOWN: in is act [pairs][n], out o float32 [pairs][cols], or (direct) y float32 [tokens][cols], which is added to.
+template <typename T, int MODE>
+__global__ void __launch_bounds__(256) experts_shared_kernel(const T* __restrict__ in, int n, const T* __restrict__ w, int cols, int top,
+                                                             const int32_t* __restrict__ ids, int pairs, int act, float limit, float alpha,
+                                                             const float* __restrict__ wts, void* __restrict__ out, int direct) {
+    extern __shared__ __align__(16) unsigned char es_sm[];
+    T* rows = reinterpret_cast<T*>(es_sm);              // [ES_PAIRS][n]
+    __shared__ int list[ES_MAX_PAIRS], counts[8];
+    dependency_wait();
+    let_dependents_start();
+    const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const bool mine = tid < pairs && ids[tid] == e;
+    const unsigned votes = __ballot_sync(0xffffffffu, mine);
+    if (lane == 0) counts[warp] = __popc(votes);
+    __syncthreads();
+    int before = 0, total = 0;
+#pragma unroll
+    for (int i = 0; i < 8; i++) { before += i < warp ? counts[i] : 0; total += counts[i]; }
+    if (total == 0) return;                             // the same for the whole block
+    if (mine) list[before + __popc(votes & ((1u << lane) - 1))] = tid;
+    constexpr int V = Vec16<T>::N, COLS = MODE == ES_GATED ? ES_STREAMS / 2 : ES_STREAMS;
+    const int c0 = (blockIdx.y * 8 + warp) * COLS;
+    const T* we = w + (size_t)e * cols * n * (MODE == ES_GATED ? 2 : 1);
+    const T* ws[ES_STREAMS];
+#pragma unroll
+    for (int s = 0; s < ES_STREAMS; s++) {
+        const int c = min(c0 + s % COLS, cols - 1);     // a column past the end: read, not written
+        ws[s] = we + ((size_t)c + (s >= COLS ? cols : 0)) * n;
+    }
+    for (int p0 = 0; p0 < total; p0 += ES_PAIRS) {
+        const int np = min(ES_PAIRS, total - p0);
+        __syncthreads();
+        for (int i = tid * V; i < np * n; i += 256 * V) {
+            const int p = i / n, d = i - p * n, pair = list[p0 + p];
+            *reinterpret_cast<uint4*>(rows + i) = *reinterpret_cast<const uint4*>(in + (size_t)(MODE == ES_DOWN ? pair : pair / top) * n + d);
+        }
+        __syncthreads();
+        if (c0 >= cols) continue;
+        float acc[ES_PAIRS][ES_STREAMS];
+        if (np == 1) es_dots<T, 1>(ws, rows, n, lane, acc);
+        else if (np == 2) es_dots<T, 2>(ws, rows, n, lane, acc);
+        else if (np == 3) es_dots<T, 3>(ws, rows, n, lane, acc);
+        else es_dots<T, 4>(ws, rows, n, lane, acc);
+#pragma unroll
+        for (int p = 0; p < ES_PAIRS; p++) {
+            if (p >= np) break;
+            const int pair = list[p0 + p];
+#pragma unroll
+            for (int s = 0; s < COLS; s++) {
+                const int c = c0 + s;
+                if (lane != p * COLS + s || c >= cols) continue;        // every lane has every sum: the lanes share the epilogue out
+                if (MODE == ES_DOWN) {
+                    if (direct) {
+                        float* y = reinterpret_cast<float*>(out) + (size_t)pair * cols + c;
+                        *y = __fadd_rn(*y, __fmul_rn(wts[pair], acc[p][s]));     // rounded as the other forms round it
+                    }
+                    else reinterpret_cast<float*>(out)[(size_t)pair * cols + c] = acc[p][s];
+                } else {
+                    float r;
+                    if (MODE == ES_UP) {
+                        r = activate_dense(act, acc[p][s]);
+                    } else if (act == 4) {
+                        const float g = fminf(acc[p][s], limit), u = fminf(fmaxf(acc[p][s + COLS], -limit), limit);
+                        r = (g / (1.0f + expf(-alpha * g))) * (u + 1.0f);
+                    } else {
+                        r = activate_rt(act, acc[p][s]) * acc[p][s + COLS];
+                    }
+                    reinterpret_cast<T*>(out)[(size_t)pair * cols + c] = from_f32<T>(r);
+                }
+            }
+        }
+    }
+}
+
 constexpr int EXPERT_TILE = 128;                        // rows of a tile of the grouped products
 
 __global__ void __launch_bounds__(1024) experts_sort_kernel(const int32_t* __restrict__ ids, int n, int E, int rows_max, int32_t* __restrict__ pos,
@@ -377,7 +489,7 @@ __global__ void __launch_bounds__(256) experts_combine_kernel(const float* __res
             float4 sum = *reinterpret_cast<const float4*>(y + (size_t)t * width + c);
             float4 total = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             for (int k = 0; k < top; k++) {
-                const int r = pos[(size_t)t * top + k];
+                const int r = pos ? pos[(size_t)t * top + k] : (ids[(size_t)t * top + k] < E ? t * top + k : -1);
                 const float w = wts[(size_t)t * top + k];
                 float4 v;
                 if (r >= 0) {
@@ -398,7 +510,7 @@ __global__ void __launch_bounds__(256) experts_combine_kernel(const float* __res
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float total = 0.0f;
         for (int k = 0; k < top; k++) {
-            const int r = pos[(size_t)t * top + k];
+            const int r = pos ? pos[(size_t)t * top + k] : (ids[(size_t)t * top + k] < E ? t * top + k : -1);
             if (r >= 0) total = fmaf(wts[(size_t)t * top + k], o[(size_t)r * width + c], total);
             else if (ids[(size_t)t * top + k] >= E) total = fmaf(wts[(size_t)t * top + k], to_f32<T>(x[(size_t)t * width + c]), total);
         }
@@ -436,7 +548,7 @@ VK_API int vk_experts_gather(const void* x, int width, const int32_t* row_token,
                             (__nv_bfloat16*)xs);
 }
 
-// y float32 [tokens][width] += sum_k wts[t][k] o[pos[t][k]]; o float32 [rows][width]; ids of E and more: the token's row of x [tokens][width].
+// pos null: a token's rows of o are t * top + k.  y float32 [tokens][width] += sum_k wts[t][k] o[pos[t][k]]; o float32 [rows][width]; ids of E and more: the token's row of x [tokens][width].
 VK_API int vk_experts_combine(const float* o, int width, int top, const int32_t* pos, const float* wts, float* y, int E, const int32_t* ids, const void* x,
                               int tokens, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VK_OK;
@@ -481,6 +593,55 @@ VK_API int vk_experts_route(const void* x, int width, const float* wr, const flo
     if (dtype == 0) return launch_dependent(experts_route_kernel<float>, dim3(tokens), dim3(128), smem, stream, (const float*)x, width, wr, br, E, top, ids, wts);
     return launch_dependent(experts_route_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), smem, stream, (const __nv_bfloat16*)x, width, wr, br, E, top,
                             ids, wts);
+}
+
+// Whether the kernels for tokens that share experts take these sizes (the launchers below refuse the others).
+VK_API int vk_experts_shared_takes(int pairs, int width, int ff, int dtype) {
+    const int v = dtype == 0 ? 4 : 8, size = dtype == 0 ? 4 : 2, longest = width > ff ? width : ff;
+    return pairs > 0 && pairs <= ES_MAX_PAIRS && width % v == 0 && ff % v == 0 && (size_t)ES_PAIRS * longest * size <= 200 * 1024;
+}
+
+template <typename T, int MODE>
+static int launch_shared(const void* in, int n, const void* w, int cols, int top, const int32_t* ids, int pairs, int E, int act, float limit, float alpha,
+                         const float* wts, void* out, int direct, cudaStream_t stream) {
+    auto kern = experts_shared_kernel<T, MODE>;
+    const size_t smem = (size_t)ES_PAIRS * n * sizeof(T);
+    if (smem > 40 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    constexpr int COLS = 8 * (MODE == ES_GATED ? ES_STREAMS / 2 : ES_STREAMS);
+    const dim3 grid(E, (cols + COLS - 1) / COLS);
+    if (grid.y > 65535) return VK_TOO_LARGE;
+    return launch_dependent(kern, grid, dim3(256), smem, stream, (const T*)in, n, (const T*)w, cols, top, ids, pairs, act, limit, alpha, wts, out, direct);
+}
+
+// vk_experts_gate_up for up to 256 (token, k) pairs.
+VK_API int vk_experts_shared_up(const void* x, int width, const void* wgu, int ff, int top, const int32_t* ids, int E, int gated, int act, float limit,
+                                float alpha, void* out, int tokens, int dtype, cudaStream_t stream) {
+    if (tokens <= 0) return VK_OK;
+    if (width <= 0 || ff <= 0 || top <= 0 || E <= 0 || act < 0 || act > 4 || (gated && act == 4 && !(limit > 0.0f))) return VK_BAD_SHAPE;
+    if (!vk_experts_shared_takes(tokens * top, width, ff, dtype)) return VK_BAD_SHAPE;
+    if (((uintptr_t)x % 16) || ((uintptr_t)wgu % 16)) return VK_BAD_ALIGNMENT;
+    const int pairs = tokens * top;
+#define VK_ES(T, MODE) return launch_shared<T, MODE>(x, width, wgu, ff, top, ids, pairs, E, act, limit, alpha, nullptr, out, 0, stream)
+    if (dtype == 0) { if (gated) VK_ES(float, ES_GATED); VK_ES(float, ES_UP); }
+    if (gated) VK_ES(__nv_bfloat16, ES_GATED);
+    VK_ES(__nv_bfloat16, ES_UP);
+#undef VK_ES
+}
+
+// act [tokens * top][ff] and wd [E][width][ff] in dtype.  direct 0: out float32 [tokens * top][width], a row a pair (vk_experts_combine follows);
+// direct 1 (top 1, no identities): out is y float32 [tokens][width], and wts[t] times the row is added to it.
+VK_API int vk_experts_shared_down(const void* act, int ff, const void* wd, int width, int top, const int32_t* ids, const float* wts, float* out, int E,
+                                  int direct, int tokens, int dtype, cudaStream_t stream) {
+    if (tokens <= 0) return VK_OK;
+    if (width <= 0 || ff <= 0 || top <= 0 || E <= 0 || (direct && top != 1)) return VK_BAD_SHAPE;
+    if (!vk_experts_shared_takes(tokens * top, width, ff, dtype)) return VK_BAD_SHAPE;
+    if (((uintptr_t)act % 16) || ((uintptr_t)wd % 16)) return VK_BAD_ALIGNMENT;
+    const int pairs = tokens * top;
+    if (dtype == 0) return launch_shared<float, ES_DOWN>(act, ff, wd, width, top, ids, pairs, E, 0, 0.0f, 0.0f, wts, out, direct, stream);
+    return launch_shared<__nv_bfloat16, ES_DOWN>(act, ff, wd, width, top, ids, pairs, E, 0, 0.0f, 0.0f, wts, out, direct, stream);
 }
 
 // tokens int32 [n_tokens] (token ids); table int32 [vocab][table_top], table_top >= top; ids int32 [n_tokens][top], wts float32 [n_tokens][top].

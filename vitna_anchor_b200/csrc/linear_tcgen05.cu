@@ -402,6 +402,9 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
     const int out_cols = EPI == TC_SWIGLU ? ex.inter : N;
     const int tiles_m = (M + TC_BM - 1) / TC_BM, tiles_n = (out_cols + tile_cols - 1) / tile_cols;
     const int num_tiles = tiles_m * tiles_n;      // tile t: rows (t % tiles_m) * 128, columns (t / tiles_m) * tile_cols
+    // Groups of rows with a weight matrix each (TcExtra): the group of a tile's rows (negative: no rows, every warp passes the tile by); a walk asks for
+    // the next tile's group before it works on the current one.
+    auto group_of = [&](int t) { return ex.tile_group && t < num_tiles ? ex.tile_group[t % tiles_m] : 0; };
 
     if (threadIdx.x == 0) {
         failed = 0;
@@ -423,8 +426,12 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
         if (lane == 0) {
             int kc = 0;                            // stages filled so far, over all of this block's tiles
             bool ok = true;
+            int g_next = group_of(blockIdx.x);
             for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
-                const int m0 = (t % tiles_m) * TC_BM, n0 = (t / tiles_m) * tile_cols;
+                const int g = g_next;
+                g_next = group_of(t + gridDim.x);
+                if (g < 0) continue;
+                const int m0 = (t % tiles_m) * TC_BM, n0 = (t / tiles_m) * tile_cols, w0 = g * ex.group_rows + n0;
                 for (int kb = 0; kb < num_kb; kb++, kc++) {
                     const int s = kc % TW_STAGES;
                     if (kc >= TW_STAGES && !mbar_wait(&empty[s], ((kc / TW_STAGES) - 1) & 1, wc.cycles)) { give_up(wc.error, &failed, 31); ok = false; break; }
@@ -432,10 +439,10 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
                     mbar_expect_tx(&full[s], STAGE_BYTES);
                     tma_load_2d(smem + s * STAGE_BYTES, &map_x, kb * TC_BK, m0, &full[s]);
                     if (EPI == TC_SWIGLU) {        // the map's box is 128 rows: gate rows, then the same rows of up
-                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, n0, &full[s]);
-                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES + B_BYTES / 2, &map_w, kb * TC_BK, ex.inter + n0, &full[s]);
+                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, w0, &full[s]);
+                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES + B_BYTES / 2, &map_w, kb * TC_BK, ex.inter + w0, &full[s]);
                     } else {
-                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, n0, &full[s]);
+                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, w0, &full[s]);
                     }
                 }
             }
@@ -446,7 +453,11 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
             const uint32_t a_lo0 = umma_desc_lo(smem_u32(smem));      // low words of the descriptors (see umma_bf16_lo)
             int kc = 0, j = 0;
             bool ok = true;
-            for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x, j++) {
+            int g_next = group_of(blockIdx.x);
+            for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
+                const int g = g_next;
+                g_next = group_of(t + gridDim.x);
+                if (g < 0) continue;
                 const int b = j & 1;
                 if (j >= 2 && !mbar_wait(&acc_empty[b], ((j >> 1) - 1) & 1, wc.cycles)) { give_up(wc.error, &failed, 32); break; }
                 tc_fence_after();
@@ -460,6 +471,7 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
                     umma_commit(&empty[s]);
                 }
                 if (ok) umma_commit(&acc_full[b]);
+                j++;
             }
         }
     } else {
@@ -469,7 +481,11 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
         const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
         int j = 0;
         bool ok = true;
-        for (int t = blockIdx.x; t < num_tiles; t += gridDim.x, j++) {
+        int g_next = group_of(blockIdx.x);
+        for (int t = blockIdx.x; t < num_tiles; t += gridDim.x) {
+            const int g = g_next;
+            g_next = group_of(t + gridDim.x);
+            if (g < 0) continue;
             const int b = j & 1;
             const int row = (t % tiles_m) * TC_BM + quarter * 32 + lane, n0 = (t / tiles_m) * tile_cols;
             if (ok && !__all_sync(0xffffffffu, mbar_wait(&acc_full[b], (j >> 1) & 1, wc.cycles))) { if (lane == 0) give_up(wc.error, &failed, 34); ok = false; }
@@ -663,6 +679,7 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
             }
             __syncwarp();
             if (lane == 0) mbar_arrive_plain(&acc_empty[b]);      // kept even after a failed wait: nobody waits for this warp without a limit
+            j++;
         }
     }
     tc_fence_before();
@@ -741,6 +758,20 @@ static bool wide_takes(int M, int out_cols, int K, int tile_cols = TW_BN) {
     if (M < 512 || out_cols < 1024 || K < 512) return false;
     const long long tiles = (long long)((M + TC_BM - 1) / TC_BM) * ((out_cols + tile_cols - 1) / tile_cols);
     return K >= 2048 || tiles * 4 >= (long long)sm_count() * 5;
+}
+
+// The same for products of row groups: M counts rows that no group fills too.  Their weights differ from tile to tile, so the second-level cache's
+// traffic bounds the narrow tiles sooner.  VITNA_GROUPED_WIDE=0 or 1 overrides (for measurements).
+static bool grouped_wide_takes(int M, int out_cols, int K) {
+    static int forced = -1;
+    if (forced < 0) {
+        const char* e = getenv("VITNA_GROUPED_WIDE");
+        forced = e ? (e[0] == '1' ? 1 : 0) : 2;
+    }
+    if (forced != 2) return forced == 1;
+    if (out_cols < 512 || K < 512) return false;
+    const long long tiles = (long long)((M + TC_BM - 1) / TC_BM) * ((out_cols + TW_BN - 1) / TW_BN);
+    return tiles >= sm_count();
 }
 
 template <int EPI, int HD = 0, int BNW = TW_BN>
@@ -869,6 +900,19 @@ VK_API int vk_linear_tcgen05_grouped(const void* x, const void* w, void* out, in
     TcExtra ex{};
     ex.tile_group = tile_group;
     ex.act = act;
+    if (grouped_wide_takes(M, N, K)) {
+        if (!make_map(&mx, x, M, K, ldx, TC_BM)) return VK_BAD_SHAPE;
+        if (gated) {
+            ex.inter = N;
+            ex.group_rows = 2 * N;
+            if (!make_map(&mw, w, groups * 2 * N, K, K, TW_BN / 2)) return VK_BAD_SHAPE;
+            return launch_wide<TC_SWIGLU>(mx, mw, out, M, 2 * N, K, error, stream, ex);
+        }
+        ex.group_rows = N;
+        if (!make_map(&mw, w, groups * N, K, K, TW_BN)) return VK_BAD_SHAPE;
+        if (mode == 0) return launch_wide<TC_SAME>(mx, mw, out, M, N, K, error, stream, ex);
+        return launch_wide<TC_F32>(mx, mw, out, M, N, K, error, stream, ex);
+    }
     if (gated) {
         ex.inter = N;
         ex.group_rows = 2 * N;

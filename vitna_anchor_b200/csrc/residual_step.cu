@@ -183,27 +183,16 @@ __global__ void __launch_bounds__(256) token_gate_kernel(const float* __restrict
 
 constexpr int TS_BLOCKS = 8, TS_THREADS = 256, TS_WARPS = TS_THREADS / 32;
 
-// Dot product of a row of T with float32 values in shared memory, the whole warp on one row; vec: 16-byte pieces.
+// Dot product of a row of T with float32 values in shared memory, the whole warp on one row.
 template <typename T>
-__device__ __forceinline__ float ts_dot(const T* __restrict__ w, const float* s, int n, int lane, bool vec) {
+__device__ __forceinline__ float ts_dot(const T* __restrict__ w, const float* s, int n, int lane) {
     float acc = 0.0f;
-    if (vec) {
-        constexpr int V = Vec16<T>::N;
-#pragma unroll 4
-        for (int i = lane * V; i < n; i += 32 * V) {
-            float f[V];
-            load16<T>(w + i, f);
-#pragma unroll
-            for (int e = 0; e < V; e += 4) {
-                const float4 x4 = *reinterpret_cast<const float4*>(s + i + e);
-                acc = fmaf(x4.x, f[e], acc); acc = fmaf(x4.y, f[e + 1], acc); acc = fmaf(x4.z, f[e + 2], acc); acc = fmaf(x4.w, f[e + 3], acc);
-            }
-        }
-    } else {
-        for (int i = lane; i < n; i += 32) acc = fmaf(s[i], to_f32<T>(w[i]), acc);
-    }
+    for (int i = lane; i < n; i += 32) acc = fmaf(s[i], to_f32<T>(w[i]), acc);
     return warp_sum(acc);
 }
+
+constexpr int TS_ROWS = 4;      // rows of the first product that a warp reads side by side
+constexpr int TS_AHEAD = 8;     // pieces of the second product's rows on their way together
 
 template <typename T>
 struct SideArgs {
@@ -241,43 +230,97 @@ __global__ void __launch_bounds__(TS_THREADS) token_side_kernel(const StepArgs<T
     let_dependents_start();
     const size_t base = (size_t)t * n;
     const int id = rs_id(a.ids, t, a.vocab);
-    for (int i = tid; i < n; i += TS_THREADS) {
-        float v = a.x[base + i];
-        if (a.c) v = fmaf(a.c[i], a.y[base + i], v);
-        xs[i] = v;
+    if (n % 4 == 0 && n4 == n && ((uintptr_t)a.x % 16) == 0 && ((uintptr_t)a.y % 16) == 0 && ((uintptr_t)a.c % 16) == 0) {
+#pragma unroll 2
+        for (int i = tid * 4; i < n; i += TS_THREADS * 4) {
+            float4 v = *reinterpret_cast<const float4*>(a.x + base + i);
+            if (a.c) {
+                const float4 y4 = *reinterpret_cast<const float4*>(a.y + base + i), c4 = *reinterpret_cast<const float4*>(a.c + i);
+                v.x = fmaf(c4.x, y4.x, v.x); v.y = fmaf(c4.y, y4.y, v.y); v.z = fmaf(c4.z, y4.z, v.z); v.w = fmaf(c4.w, y4.w, v.w);
+            }
+            *reinterpret_cast<float4*>(xs + i) = v;
+        }
+    } else {
+        for (int i = tid; i < n; i += TS_THREADS) {
+            float v = a.x[base + i];
+            if (a.c) v = fmaf(a.c[i], a.y[base + i], v);
+            xs[i] = v;
+        }
     }
     __syncthreads();
     // a's rows, dealt out to the blocks in turn; every block gets every g
-    for (int r = warp * TS_BLOCKS + rank; r < dim; r += TS_WARPS * TS_BLOCKS) {
-        const float s = ts_dot<T>(sd.gate + (size_t)r * n, xs, n, lane, vec_gate);
+    constexpr int V = Vec16<T>::N, STRIDE = TS_WARPS * TS_BLOCKS;
+    auto give = [&](int r, float s) {
         const float v = rs_gelu(s) * to_f32<T>(sd.side[(size_t)id * sd.ld + sd.off + r]);
         if (lane < TS_BLOCKS) cluster.map_shared_rank(g, lane)[r] = v;
+    };
+    if (vec_gate) {
+        for (int r = warp * TS_BLOCKS + rank; r < dim; r += STRIDE * TS_ROWS) {
+            const T* w[TS_ROWS];
+            float acc[TS_ROWS];
+#pragma unroll
+            for (int q = 0; q < TS_ROWS; q++) { w[q] = sd.gate + (size_t)min(r + q * STRIDE, dim - 1) * n; acc[q] = 0.0f; }
+#pragma unroll 2
+            for (int i = lane * V; i < n; i += 32 * V) {
+                float f[TS_ROWS][V];
+#pragma unroll
+                for (int q = 0; q < TS_ROWS; q++) load16<T>(w[q] + i, f[q]);
+#pragma unroll
+                for (int e = 0; e < V; e += 4) {
+                    const float4 x4 = *reinterpret_cast<const float4*>(xs + i + e);
+#pragma unroll
+                    for (int q = 0; q < TS_ROWS; q++) {
+                        acc[q] = fmaf(x4.x, f[q][e], acc[q]); acc[q] = fmaf(x4.y, f[q][e + 1], acc[q]);
+                        acc[q] = fmaf(x4.z, f[q][e + 2], acc[q]); acc[q] = fmaf(x4.w, f[q][e + 3], acc[q]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int q = 0; q < TS_ROWS; q++) {
+                const float s = warp_sum(acc[q]);
+                if (r + q * STRIDE < dim) give(r + q * STRIDE, s);
+            }
+        }
+    } else {
+        for (int r = warp * TS_BLOCKS + rank; r < dim; r += STRIDE) give(r, ts_dot<T>(sd.gate + (size_t)r * n, xs, n, lane));
     }
     cluster.sync();
     // this block's rows of z
     float ss = 0.0f;
-    constexpr int V = Vec16<T>::N;
     if (vec_proj) {                                     // a row is dim / V pieces: several rows a warp where it is short
         int lanes = 1;
         while (lanes < 32 && lanes * V < dim) lanes *= 2;
-        const int rows = 32 / lanes, sub = lane / lanes, in = lane - sub * lanes;
-        for (int r0 = lo + warp * rows; r0 < hi; r0 += TS_WARPS * rows) {
-            const int r = r0 + sub;
-            float acc = 0.0f;
-            if (r < hi) {
-                for (int i = in * V; i < dim; i += lanes * V) {
-                    float f[V];
-                    load16<T>(sd.proj + (size_t)r * dim + i, f);
+        const int rows = 32 / lanes, sub = lane / lanes, in = lane - sub * lanes, step = TS_WARPS * rows;
+        for (int r0 = lo + warp * rows + sub; r0 - sub < hi; r0 += step * TS_AHEAD) {
+            float acc[TS_AHEAD];
 #pragma unroll
-                    for (int e = 0; e < V; e++) acc = fmaf(g[i + e], f[e], acc);
+            for (int q = 0; q < TS_AHEAD; q++) acc[q] = 0.0f;
+            for (int i = in * V; i < dim; i += lanes * V) {
+                uint4 piece[TS_AHEAD];
+#pragma unroll
+                for (int q = 0; q < TS_AHEAD; q++)
+                    piece[q] = *reinterpret_cast<const uint4*>(sd.proj + (size_t)min(r0 + q * step, hi - 1) * dim + i);
+                float gv[V];
+#pragma unroll
+                for (int e = 0; e < V; e += 4) *reinterpret_cast<float4*>(gv + e) = *reinterpret_cast<const float4*>(g + i + e);
+#pragma unroll
+                for (int q = 0; q < TS_AHEAD; q++) {
+                    float f[V];
+                    load16<T>(reinterpret_cast<const T*>(&piece[q]), f);
+#pragma unroll
+                    for (int e = 0; e < V; e++) acc[q] = fmaf(gv[e], f[e], acc[q]);
                 }
             }
-            for (int o = lanes / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-            if (r < hi && in == 0) zs[r - lo] = acc;
+#pragma unroll
+            for (int q = 0; q < TS_AHEAD; q++) {
+                for (int o = lanes / 2; o > 0; o >>= 1) acc[q] += __shfl_xor_sync(0xffffffffu, acc[q], o);
+                const int r = r0 + q * step;
+                if (r < hi && in == 0) zs[r - lo] = acc[q];
+            }
         }
     } else {
         for (int r = lo + warp; r < hi; r += TS_WARPS) {
-            const float v = ts_dot<T>(sd.proj + (size_t)r * dim, g, dim, lane, false);
+            const float v = ts_dot<T>(sd.proj + (size_t)r * dim, g, dim, lane);
             if (lane == 0) zs[r - lo] = v;
         }
     }

@@ -1463,6 +1463,46 @@ def experts_apply(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor
     return y
 
 
+def experts_share(tokens: int, top: int, E: int) -> bool:
+    """Whether a step of few tokens has enough of them to an expert that reading each chosen expert once pays: the pairs against the number of
+    different experts that as many tokens choose on average."""
+    return tokens * top >= 1.25 * E * (1.0 - (1.0 - top / max(E, top)) ** tokens)
+
+
+def experts_shared_takes(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, top: int) -> bool:
+    return (bool(lib().vk_experts_shared_takes(x.shape[0] * top, x.shape[1], w_down.shape[2], _dt(x))) and x.stride(0) == x.shape[1]
+            and x.data_ptr() % 16 == 0 and w_gate_up.data_ptr() % 16 == 0 and w_down.data_ptr() % 16 == 0)
+
+
+def experts_apply_shared(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, act_buf: torch.Tensor,
+                         o: Optional[torch.Tensor], y: torch.Tensor, activation: str = "silu", limit: float = 0.0, alpha: float = 1.702,
+                         gated: bool = True) -> torch.Tensor:
+    """experts_apply for up to 256 (token, k) pairs, the same bits, with every chosen expert's rows read once for all tokens that chose it.
+    o float32 [T * top, W] is scratch (None: a token has one expert and there are no identities; the second kernel then adds to y itself)."""
+    _req(x, "x", dims=2); _req(w_gate_up, "w_gate_up", x.dtype, 3); _req(w_down, "w_down", x.dtype, 3); _req(y, "y", torch.float32, 2)
+    _req(act_buf, "act_buf", x.dtype, 2)
+    T, W = x.shape
+    E, rows, _ = w_gate_up.shape
+    per = 2 if gated else 1
+    ff, top = rows // per, ids.shape[1]
+    if w_gate_up.shape != (E, per * ff, W) or w_down.shape != (E, W, ff) or y.shape != (T, W) or act_buf.shape != (T * top, ff):
+        raise KernelError("experts_apply_shared: shapes do not fit")
+    if o is not None:
+        _req(o, "o", torch.float32, 2)
+        if o.shape != (T * top, W):
+            raise KernelError("experts_apply_shared: o is not [pairs, width]")
+    elif top != 1:
+        raise KernelError("experts_apply_shared: several experts a token need the rows between")
+    act = _expert_act(activation, "experts_apply_shared", gated)
+    _check(lib().vk_experts_shared_up(_p(x), W, _p(w_gate_up), ff, top, _p(ids), E, int(gated), act, ctypes.c_float(limit), ctypes.c_float(alpha),
+                                      _p(act_buf), T, _dt(x), _stream()), "experts_shared_up")
+    _check(lib().vk_experts_shared_down(_p(act_buf), ff, _p(w_down), W, top, _p(ids), _p(wts), _p(y if o is None else o), E, int(o is None), T, _dt(x),
+                                        _stream()), "experts_shared_down")
+    if o is not None:
+        _check(lib().vk_experts_combine(_p(o), W, top, _p(None), _p(wts), _p(y), E, _p(ids), _p(x), T, _dt(x), _stream()), "experts_combine")
+    return y
+
+
 def experts_grouped_rows(tokens: int, top: int, E: int) -> int:
     """Rows of the grouped matrix for up to `tokens` tokens: every copy, and every expert's rows filled up to whole tiles."""
     rows = int(lib().vk_experts_grouped_rows(tokens, top, E))

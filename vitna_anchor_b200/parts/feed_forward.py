@@ -136,8 +136,8 @@ class RoutedExperts(FeedForward):
     w_down [E, hidden, ff] in the compute dtype; `shared`: a FeedForward every token passes as well (or None).  The router's
     logits are float32 sums over the (compute dtype) input.  Which experts run never comes to the host: the kernels read the
     choice on the device, so the part is replayed faithfully from a graph.  Steps with at least GROUPED_FROM (token, expert) pairs in
-    bfloat16 run the experts as products of row groups on the tensor cores; shorter steps and float32 read each token's experts' rows
-    directly."""
+    bfloat16 run the experts as products of row groups on the tensor cores; shorter steps and float32 read the experts' rows
+    directly: every chosen expert's once where a few tokens share experts, else each token's."""
 
     GROUPED_FROM = 256
 
@@ -217,6 +217,13 @@ class RoutedExperts(FeedForward):
                                       None if self.activation != "clamped" else
                                       ws.flat(f"moe.gu/{key}/{self.intermediate}", rows_max * 2 * self.intermediate, ctx.dtype)[:rows * 2 * self.intermediate].view(rows, 2 * self.intermediate),
                                       gated=self.gated)
+        elif ops.experts_share(T, self.top, self.E) and ops.experts_shared_takes(xn, self.w_gate_up, self.w_down, self.top):
+            # few tokens that share experts: each chosen expert's rows are read once
+            act = ws.flat(f"moe.act/{self.top}/{self.intermediate}", ws.max_tokens * self.top * self.intermediate, ctx.dtype)
+            pairs, direct = T * self.top, self.top == 1 and (self.scored is None or not self.scored.identities)
+            o = None if direct else ws.flat(f"moe.few/{self.hidden}", 256 * self.hidden, torch.float32)[:pairs * self.hidden].view(pairs, self.hidden)
+            ops.experts_apply_shared(xn, self.w_gate_up, self.w_down, ids, wts, act[:pairs * self.intermediate].view(pairs, self.intermediate), o, residual,
+                                     self.activation, self.limit, self.alpha, self.gated)
         else:
             act = ws.flat(f"moe.act/{self.top}/{self.intermediate}", ws.max_tokens * self.top * self.intermediate, ctx.dtype)
             ops.experts_apply(xn, self.w_gate_up, self.w_down, ids, wts, act[:T * self.top * self.intermediate].view(T * self.top, self.intermediate),
