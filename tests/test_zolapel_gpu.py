@@ -447,6 +447,24 @@ def test_the_per_layer_input_in_one_kernel(sizes, dtype):
     assert np.abs(_f(got) - want).max() < (1e-5 if dtype == torch.float32 else 1e-2) * max(1.0, np.abs(want).max())
 
 
+@pytest.mark.parametrize("sizes", [(64, 12, 9), (2048, 256, 0), (96, 5, 3), (1024, 40, 24), (72, 128, 8), (42, 16, 0)])
+@pytest.mark.parametrize("T", [7, 64, 70, 300])
+def test_a_product_with_the_gate_and_the_token_s_factor_behind_it(sizes, T):
+    from vitna_anchor_b200 import ops
+    n, dim, off = sizes
+    rng = np.random.default_rng(n + T)
+    V = 17
+    for dtype in (torch.float32, torch.bfloat16):
+        x, w = _dev(rng.standard_normal((T, n)), dtype), _dev(rng.standard_normal((dim, n)) * n ** -0.5, dtype)
+        side = _dev(rng.standard_normal((V, dim + off + 8)), dtype)
+        ids = torch.from_numpy(rng.integers(0, V, T).astype(np.int32)).cuda()
+        out = torch.zeros(T, dim, dtype=dtype, device="cuda")
+        ops.linear_token_gate(x, w, side, off, ids, torch.empty(T, dim, device="cuda"), out)
+        want = PZ.gelu_tanh(_f(x) @ _f(w).T) * _f(side)[ids.cpu().numpy(), off:off + dim]
+        assert np.abs(_f(out) - want).max() < (2e-5 if dtype == torch.float32 else 2e-2) * max(1.0, np.abs(want).max()), dtype
+    ops.check_device_errors()
+
+
 @pytest.mark.parametrize("sizes", [(4, 2, 16, 16, 8), (3, 1, 96, 96, 96), (20, 4, 64, 64, 30), (5, 5, 7, 7, 2), (2, 1, 256, 256, 256), (3, 3, 12, 20, 6), (2, 2, 260, 260, 8),
                                    (1, 1, 10, 10, 0)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -213,8 +213,8 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
     auto places = [&](int j, int& a, int& b) {
         if (!neighbours && j < half) { a = j; b = j + half; } else { a = 2 * j; b = a + 1; }
     };
-    float2 v[P], ahead[2][P];                           // this head's row, and the warp's next two
-    auto fetch = [&](int h, float2* v) {
+    float2 v[P];
+    auto fetch = [&](int h) {
         const float* row = in + (size_t)h * hd;
 #pragma unroll
         for (int p = 0; p < P; p++) {
@@ -225,17 +225,14 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
             v[p] = b == a + 1 ? *reinterpret_cast<const float2*>(row + a) : make_float2(row[a], row[b]);
         }
     };
-    fetch(min(warp, n_qk - 1), v);
-    if (warp + nwarps < n_qk) fetch(warp + nwarps, ahead[0]);
-    if (warp + 2 * nwarps < n_qk) fetch(warp + 2 * nwarps, ahead[1]);
+    if (warp < n_qk) fetch(warp);
     const float pos = (float)positions[t];
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         const float ang = pos * freq[i];
         sincosf(ang, &nr_turn[2 * i + 1], &nr_turn[2 * i]);
     }
     __syncthreads();
-    int round = 0;
-    for (int h = warp; h < n_heads; h += nwarps, round++) {
+    for (int h = warp; h < n_heads; h += nwarps) {
         if (h >= n_qk) {                                // a value head of its own
             if (s < 0) continue;
             const int g = h - n_qk;
@@ -244,12 +241,7 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
             for (int d = lane; d < vd; d += 32) dst[d] = from_f32<T>(row[d] * v_mult);
             continue;
         }
-        if (round == 1 || round == 2) {
-#pragma unroll
-            for (int p = 0; p < P; p++) v[p] = round == 1 ? ahead[0][p] : ahead[1][p];
-        } else if (round > 2) {
-            fetch(h, v);
-        }
+        if (h != warp) fetch(h);
         const bool key = h >= nh;
         if (key && s < 0) continue;
         const float* w = key ? kn_w : qn_w;
@@ -281,6 +273,67 @@ __global__ void __launch_bounds__(256) normed_rotary_store_kernel(const float* _
             }
             if (b == a + 1) am_store2<T>(dst + a, x, y);
             else { dst[a] = from_f32<T>(x); dst[b] = from_f32<T>(y); }
+        }
+    }
+}
+
+// The same for pairs of neighbours where every size is a multiple of four, heads have up to 128 values and everything lies on 16 bytes (which
+// is what the tensor-core attentions take): a lane has four neighbours of a head, two whole pairs, in one 16-byte load.
+template <typename T>
+__global__ void __launch_bounds__(256) normed_neighbours_store_kernel(const float* __restrict__ proj, int N, const int32_t* __restrict__ positions,
+                                                                      const int32_t* __restrict__ slot, const float* __restrict__ qn_w,
+                                                                      const float* __restrict__ kn_w, float eps, const float* __restrict__ freq, int dims,
+                                                                      T* __restrict__ q_out, T* __restrict__ cache, int nh, int nkv, int hd, int vd,
+                                                                      int page_size, float v_mult, int v_from_k) {
+    __shared__ __align__(16) float turn[128];           // [dims/2][2] cos and sin of the token's angles
+    dependency_wait();
+    let_dependents_start();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const int n_qk = nh + nkv, n_heads = v_from_k ? n_qk : n_qk + nkv, d = lane * 4;
+    const bool on = d < hd;
+    const float* in = proj + (size_t)t * N;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 v = zero, next = zero;
+    if (on && warp < n_qk) v = *reinterpret_cast<const float4*>(in + (size_t)warp * hd + d);
+    if (on && warp + nwarps < n_qk) next = *reinterpret_cast<const float4*>(in + (size_t)(warp + nwarps) * hd + d);
+    const int s = (slot && cache) ? slot[t] : -1;
+    const float4 one = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+    const float4 wq = qn_w && on ? *reinterpret_cast<const float4*>(qn_w + d) : one, wk = kn_w && on ? *reinterpret_cast<const float4*>(kn_w + d) : one;
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < dims / 2; i += blockDim.x) sincosf(pos * freq[i], &turn[2 * i + 1], &turn[2 * i]);
+    const size_t page = s >= 0 ? (size_t)(s / page_size) : 0;
+    T* kbase = cache + page * ((size_t)nkv * page_size * (hd + vd)) + (size_t)(s >= 0 ? s % page_size : 0) * hd;
+    T* vbase = cache + page * ((size_t)nkv * page_size * (hd + vd)) + (size_t)nkv * page_size * hd + (size_t)(s >= 0 ? s % page_size : 0) * vd;
+    const float inv_n = 1.0f / (float)hd;
+    __syncthreads();
+    const float4 cs = d < dims ? *reinterpret_cast<const float4*>(turn + d) : make_float4(1.0f, 0.0f, 1.0f, 0.0f);
+    for (int h = warp; h < n_heads; h += nwarps) {
+        if (h >= n_qk) {                                // a value head of its own
+            if (s < 0) continue;
+            const int g = h - n_qk;
+            for (int e = d; e < vd; e += 128) {
+                const float4 u = *reinterpret_cast<const float4*>(in + (size_t)n_qk * hd + (size_t)g * vd + e);
+                am_store4<T>(vbase + (size_t)g * page_size * vd + e, make_float4(u.x * v_mult, u.y * v_mult, u.z * v_mult, u.w * v_mult));
+            }
+            continue;
+        }
+        const float4 u = v;
+        v = next;
+        if (on && h + 2 * nwarps < n_qk) next = *reinterpret_cast<const float4*>(in + (size_t)(h + 2 * nwarps) * hd + d);
+        const bool key = h >= nh;
+        if (key && s < 0) continue;
+        float inv = 1.0f;
+        if (eps >= 0.0f) inv = 1.0f / sqrtf(warp_sum(fmaf(u.x, u.x, u.y * u.y) + fmaf(u.z, u.z, u.w * u.w)) * inv_n + eps);
+        if (!on) continue;
+        const float4 w = key ? wk : wq;
+        const float a0 = u.x * inv * w.x, b0 = u.y * inv * w.y, a1 = u.z * inv * w.z, b1 = u.w * inv * w.w;
+        const float4 r = make_float4(a0 * cs.x - b0 * cs.y, b0 * cs.x + a0 * cs.y, a1 * cs.z - b1 * cs.w, b1 * cs.z + a1 * cs.w);
+        if (!key) {
+            am_store4<T>(q_out + ((size_t)t * nh + h) * hd + d, r);
+        } else {
+            am_store4<T>(kbase + (size_t)(h - nh) * page_size * hd + d, r);
+            if (v_from_k)
+                am_store4<T>(vbase + (size_t)(h - nh) * page_size * vd + d, make_float4(u.x * v_mult, u.y * v_mult, u.z * v_mult, u.w * v_mult));
         }
     }
 }
@@ -813,6 +866,15 @@ VK_API int vk_mixed_attn_prepare(const float* proj, int N, const int32_t* positi
     const size_t smem = (size_t)(dims + vd + 1) * sizeof(float);
     if (smem > 48 * 1024) return VK_TOO_LARGE;
     auto on16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+    if (neighbours && !vfreq && !bias && hd % 4 == 0 && hd <= 128 && vd % 4 == 0 && dims % 4 == 0 && N % 4 == 0 && on16(proj) && on16(q_out) && on16(cache) &&
+        on16(qn_w) && on16(kn_w)) {
+        const int threads = nh + nkv >= 8 ? 256 : 128;
+        if (dtype == 0)
+            return launch_dependent(normed_neighbours_store_kernel<float>, dim3(tokens), dim3(threads), 0, stream, proj, N, positions, slot, qn_w, kn_w, eps,
+                                    freq, dims, (float*)q_out, (float*)cache, nh, nkv, hd, vd, page_size, v_mult, v_from_k);
+        return launch_dependent(normed_neighbours_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream, proj, N, positions, slot, qn_w, kn_w,
+                                eps, freq, dims, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, nh, nkv, hd, vd, page_size, v_mult, v_from_k);
+    }
     auto on8 = [](const void* p) { return ((uintptr_t)p % 8) == 0; };
     if (!vfreq && !bias && (eps >= 0.0f || neighbours || v_from_k) && hd % 2 == 0 && vd % 2 == 0 && hd <= 256 && N % 2 == 0 && on8(proj) && on8(q_out) && on8(cache)) {
         if (dtype == 0)

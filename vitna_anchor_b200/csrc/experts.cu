@@ -88,7 +88,7 @@ __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict_
 
 // A block TB tokens (a row of the router is read once for all of them); a warp a logit, then a warp a token.  all = experts + identities.
 template <typename T, int TB>
-__global__ void __launch_bounds__(256) experts_route_scored_kernel(const T* __restrict__ x, int width, const float* __restrict__ wr,
+__global__ void __launch_bounds__(TB == 1 ? 1024 : 256) experts_route_scored_kernel(const T* __restrict__ x, int width, const float* __restrict__ wr,
                                                                    const float* __restrict__ correction, int all, int top, int count, int keep, float scale,
                                                                    int32_t* __restrict__ ids, float* __restrict__ wts, int tokens, int vec, int sigmoid,
                                                                    int squared) {
@@ -571,8 +571,10 @@ VK_API int vk_experts_route_scored(const void* x, int width, const float* wr, co
     if (smem > 48 * 1024) return VK_TOO_LARGE;
     const dim3 grid((tokens + tb - 1) / tb);
     const int vec = width % (dtype == 0 ? 4 : 8) == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)wr % 16) == 0;
+    int warps = tb == 1 && all > 8 ? all : 8;           // few tokens: a warp a logit, as far as a block has warps
+    if (warps > 32) warps = 32;
 #define VK_ERS(T, TB)                                                                                                                          \
-    return launch_dependent(experts_route_scored_kernel<T, TB>, grid, dim3(256), smem, stream, (const T*)x, width, wr, correction, all, top, count, \
+    return launch_dependent(experts_route_scored_kernel<T, TB>, grid, dim3(32 * warps), smem, stream, (const T*)x, width, wr, correction, all, top, count, \
                             keep, scale, ids, wts, tokens, vec, sigmoid, squared)
     if (dtype == 0) {
         if (tb == 4) VK_ERS(float, 4);

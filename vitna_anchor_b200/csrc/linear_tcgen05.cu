@@ -21,7 +21,7 @@ namespace vk {
 
 constexpr int TC_BM = 128, TC_BK = 64, TC_THREADS = 192;
 template <int BN> struct TcStages { static constexpr int N = BN >= 128 ? 3 : 4; };   // 96 KB of stages either way: two blocks a multiprocessor
-enum { TC_SAME = 0, TC_F32 = 1, TC_ACC = 2, TC_SWIGLU = 3, TC_ROPE = 4 };
+enum { TC_SAME = 0, TC_F32 = 1, TC_ACC = 2, TC_SWIGLU = 3, TC_ROPE = 4, TC_TOKEN = 5 };
 
 // What the fused epilogues need besides the accumulator.
 //   TC_SWIGLU  the weight is [2*inter, K], gate rows then up rows; a block's tile is 64 gate rows and the 64 up rows
@@ -30,6 +30,7 @@ enum { TC_SAME = 0, TC_F32 = 1, TC_ACC = 2, TC_SWIGLU = 3, TC_ROPE = 4 };
 //   TC_ROPE    the weight is [(nh + 2*nkv) * hd, K]; BN = hd, so a tile is one head: a q head is rotated by the
 //              token's position and written to out [M, nh*hd]; a k head is rotated and written into the token's
 //              cache slot; a v head is written there as it is (engine/src/ops.c:273-281, engine/src/model.c:927-930)
+//   TC_TOKEN   a row belongs to a token: out (bfloat16) = gelu(sum) in its tanh form times the token's row of a table, columns tok_off ..
 // silu(g) * up for the bfloat16 path: 2^x and the reciprocal come from the special-function unit (relative error about
 // 1e-6, far below the bfloat16 rounding of the result); the float32 path keeps expf and the division.
 __device__ __forceinline__ float tc_silu_mul(float g, float up) {
@@ -53,6 +54,9 @@ struct TcExtra {
     // blocks leave at once).  The table is the output of a kernel before this one.  Null: one weight matrix for all rows.
     const int32_t* tile_group;
     int group_rows;
+    const __nv_bfloat16* tok_table;      // TC_TOKEN: [tok_vocab][tok_ld]
+    const int32_t* tok_ids;
+    int tok_ld, tok_off, tok_vocab;
 };
 
 template <int BN, int EPI>
@@ -309,6 +313,30 @@ __global__ void __launch_bounds__(TC_THREADS) linear_tcgen05_kernel(const __grid
                 const bool whole = col + 32 <= N;
                 if (row >= M || col >= N) {
                     // nothing of this thread's to store
+                } else if (EPI == TC_TOKEN) {
+                    int id = ex.tok_ids[row];
+                    if (id < 0 || id >= ex.tok_vocab) id = 0;           // the host has checked the range; never read outside the table
+                    const __nv_bfloat16* e = ex.tok_table + (size_t)id * ex.tok_ld + ex.tok_off + col;
+                    __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * N + col;
+                    if (whole && (N % 8 == 0) && ((reinterpret_cast<uintptr_t>(e) % 16) == 0)) {
+#pragma unroll
+                        for (int j = 0; j < 32; j += 8) {
+                            float f[8];
+                            load16<__nv_bfloat16>(e + j, f);
+                            uint32_t p[4];
+#pragma unroll
+                            for (int q = 0; q < 8; q += 2) {
+                                __nv_bfloat162 v = __floats2bfloat162_rn(activate_rt(2, __uint_as_float(r[j + q])) * f[q],
+                                                                         activate_rt(2, __uint_as_float(r[j + q + 1])) * f[q + 1]);
+                                p[q / 2] = *reinterpret_cast<uint32_t*>(&v);
+                            }
+                            *reinterpret_cast<uint4*>(o + j) = make_uint4(p[0], p[1], p[2], p[3]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 32; j++)
+                            if (col + j < N) o[j] = __float2bfloat16_rn(activate_rt(2, __uint_as_float(r[j])) * __bfloat162float(e[j]));
+                    }
                 } else if (EPI == TC_SAME) {
                     __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * N + col;
                     if (ex.act) {
@@ -402,9 +430,6 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
     const int out_cols = EPI == TC_SWIGLU ? ex.inter : N;
     const int tiles_m = (M + TC_BM - 1) / TC_BM, tiles_n = (out_cols + tile_cols - 1) / tile_cols;
     const int num_tiles = tiles_m * tiles_n;      // tile t: rows (t % tiles_m) * 128, columns (t / tiles_m) * tile_cols
-    // Groups of rows with a weight matrix each (TcExtra): the group of a tile's rows (negative: no rows, every warp passes the tile by); a walk asks for
-    // the next tile's group before it works on the current one.
-    auto group_of = [&](int t) { return ex.tile_group && t < num_tiles ? ex.tile_group[t % tiles_m] : 0; };
 
     if (threadIdx.x == 0) {
         failed = 0;
@@ -426,12 +451,8 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
         if (lane == 0) {
             int kc = 0;                            // stages filled so far, over all of this block's tiles
             bool ok = true;
-            int g_next = group_of(blockIdx.x);
             for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
-                const int g = g_next;
-                g_next = group_of(t + gridDim.x);
-                if (g < 0) continue;
-                const int m0 = (t % tiles_m) * TC_BM, n0 = (t / tiles_m) * tile_cols, w0 = g * ex.group_rows + n0;
+                const int m0 = (t % tiles_m) * TC_BM, n0 = (t / tiles_m) * tile_cols;
                 for (int kb = 0; kb < num_kb; kb++, kc++) {
                     const int s = kc % TW_STAGES;
                     if (kc >= TW_STAGES && !mbar_wait(&empty[s], ((kc / TW_STAGES) - 1) & 1, wc.cycles)) { give_up(wc.error, &failed, 31); ok = false; break; }
@@ -439,10 +460,10 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
                     mbar_expect_tx(&full[s], STAGE_BYTES);
                     tma_load_2d(smem + s * STAGE_BYTES, &map_x, kb * TC_BK, m0, &full[s]);
                     if (EPI == TC_SWIGLU) {        // the map's box is 128 rows: gate rows, then the same rows of up
-                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, w0, &full[s]);
-                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES + B_BYTES / 2, &map_w, kb * TC_BK, ex.inter + w0, &full[s]);
+                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, n0, &full[s]);
+                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES + B_BYTES / 2, &map_w, kb * TC_BK, ex.inter + n0, &full[s]);
                     } else {
-                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, w0, &full[s]);
+                        tma_load_2d(smem + s * STAGE_BYTES + A_BYTES, &map_w, kb * TC_BK, n0, &full[s]);
                     }
                 }
             }
@@ -453,11 +474,7 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
             const uint32_t a_lo0 = umma_desc_lo(smem_u32(smem));      // low words of the descriptors (see umma_bf16_lo)
             int kc = 0, j = 0;
             bool ok = true;
-            int g_next = group_of(blockIdx.x);
-            for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
-                const int g = g_next;
-                g_next = group_of(t + gridDim.x);
-                if (g < 0) continue;
+            for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x, j++) {
                 const int b = j & 1;
                 if (j >= 2 && !mbar_wait(&acc_empty[b], ((j >> 1) - 1) & 1, wc.cycles)) { give_up(wc.error, &failed, 32); break; }
                 tc_fence_after();
@@ -471,7 +488,6 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
                     umma_commit(&empty[s]);
                 }
                 if (ok) umma_commit(&acc_full[b]);
-                j++;
             }
         }
     } else {
@@ -481,11 +497,7 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
         const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
         int j = 0;
         bool ok = true;
-        int g_next = group_of(blockIdx.x);
-        for (int t = blockIdx.x; t < num_tiles; t += gridDim.x) {
-            const int g = g_next;
-            g_next = group_of(t + gridDim.x);
-            if (g < 0) continue;
+        for (int t = blockIdx.x; t < num_tiles; t += gridDim.x, j++) {
             const int b = j & 1;
             const int row = (t % tiles_m) * TC_BM + quarter * 32 + lane, n0 = (t / tiles_m) * tile_cols;
             if (ok && !__all_sync(0xffffffffu, mbar_wait(&acc_full[b], (j >> 1) & 1, wc.cycles))) { if (lane == 0) give_up(wc.error, &failed, 34); ok = false; }
@@ -679,7 +691,6 @@ __global__ void __launch_bounds__(TW_THREADS, 1) linear_tcgen05_wide_kernel(cons
             }
             __syncwarp();
             if (lane == 0) mbar_arrive_plain(&acc_empty[b]);      // kept even after a failed wait: nobody waits for this warp without a limit
-            j++;
         }
     }
     tc_fence_before();
@@ -760,20 +771,6 @@ static bool wide_takes(int M, int out_cols, int K, int tile_cols = TW_BN) {
     return K >= 2048 || tiles * 4 >= (long long)sm_count() * 5;
 }
 
-// The same for products of row groups: M counts rows that no group fills too.  Their weights differ from tile to tile, so the second-level cache's
-// traffic bounds the narrow tiles sooner.  VITNA_GROUPED_WIDE=0 or 1 overrides (for measurements).
-static bool grouped_wide_takes(int M, int out_cols, int K) {
-    static int forced = -1;
-    if (forced < 0) {
-        const char* e = getenv("VITNA_GROUPED_WIDE");
-        forced = e ? (e[0] == '1' ? 1 : 0) : 2;
-    }
-    if (forced != 2) return forced == 1;
-    if (out_cols < 512 || K < 512) return false;
-    const long long tiles = (long long)((M + TC_BM - 1) / TC_BM) * ((out_cols + TW_BN - 1) / TW_BN);
-    return tiles >= sm_count();
-}
-
 template <int EPI, int HD = 0, int BNW = TW_BN>
 static int launch_wide(const CUtensorMap& mx, const CUtensorMap& mw, void* out, int M, int N, int K, int* error, cudaStream_t stream,
                        const TcExtra& ex = TcExtra{}) {
@@ -811,6 +808,14 @@ static int linear_tcgen05_impl(const void* x, const void* w, void* out, int M, i
     if ((M + TC_BM - 1) / TC_BM > 65535) return VK_TOO_LARGE;
     if (wide_takes(M, N, K)) {
         CUtensorMap wx, ww;
+        // tiles of 192 columns where a block's rounds of them are shorter than its rounds of 256 (see the gated form)
+        const long long tiles_m = (M + TC_BM - 1) / TC_BM, sms = sm_count();
+        const long long rounds256 = (tiles_m * ((N + 255) / 256) + sms - 1) / sms, rounds192 = (tiles_m * ((N + 191) / 192) + sms - 1) / sms;
+        if (mode != 2 && rounds192 * 192 < rounds256 * 256) {
+            if (!make_map(&wx, x, M, K, ldx, TC_BM) || !make_map(&ww, w, N, K, K, 192)) return VK_BAD_SHAPE;
+            if (mode == 0) return launch_wide<TC_SAME, 0, 192>(wx, ww, out, M, N, K, error, stream, ex);
+            return launch_wide<TC_F32, 0, 192>(wx, ww, out, M, N, K, error, stream);
+        }
         if (!make_map(&wx, x, M, K, ldx, TC_BM) || !make_map(&ww, w, N, K, K, TW_BN)) return VK_BAD_SHAPE;
         if (mode == 0) return launch_wide<TC_SAME>(wx, ww, out, M, N, K, error, stream, ex);
         if (mode == 1) return launch_wide<TC_F32>(wx, ww, out, M, N, K, error, stream);
@@ -839,6 +844,22 @@ VK_API int vk_linear_tcgen05(const void* x, const void* w, void* out, int M, int
 VK_API int vk_linear_tcgen05_act(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int act, int* error,
                                  cudaStream_t stream) {
     return linear_tcgen05_impl(x, w, out, M, N, K, ldx, 0, act, error, stream);
+}
+
+// out [M, N] (bfloat16) = gelu(x @ w.T) (the tanh form) times row ids[m] of table [vocab][ld] (bfloat16), columns off .. off + N.
+VK_API int vk_linear_tcgen05_token(const void* x, const void* w, void* out, int M, int N, int K, int ldx, const void* table, int ld, int off,
+                                   const int32_t* ids, int vocab, int* error, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return VK_OK;
+    if (K <= 0 || ldx < K || !error || !table || !ids || vocab <= 0 || off < 0 || off + N > ld || K % 8 != 0 || ldx % 8 != 0) return VK_BAD_SHAPE;
+    if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || ((uintptr_t)out % 16)) return VK_BAD_ALIGNMENT;
+    if ((M + TC_BM - 1) / TC_BM > 65535) return VK_TOO_LARGE;
+    TcExtra ex{};
+    ex.tok_table = (const __nv_bfloat16*)table;
+    ex.tok_ids = ids;
+    ex.tok_ld = ld; ex.tok_off = off; ex.tok_vocab = vocab;
+    CUtensorMap mx, mw;
+    if (!make_map(&mx, x, M, K, ldx, TC_BM) || !make_map(&mw, w, N, K, K, 32)) return VK_BAD_SHAPE;
+    return launch_tc<32, TC_TOKEN>(mx, mw, out, M, N, K, error, stream, ex);
 }
 
 // x [M, K] bfloat16 (row stride ldx), w [2*inter, K] bfloat16 with gate rows then up rows, out [M, inter] bfloat16 =
@@ -900,19 +921,6 @@ VK_API int vk_linear_tcgen05_grouped(const void* x, const void* w, void* out, in
     TcExtra ex{};
     ex.tile_group = tile_group;
     ex.act = act;
-    if (grouped_wide_takes(M, N, K)) {
-        if (!make_map(&mx, x, M, K, ldx, TC_BM)) return VK_BAD_SHAPE;
-        if (gated) {
-            ex.inter = N;
-            ex.group_rows = 2 * N;
-            if (!make_map(&mw, w, groups * 2 * N, K, K, TW_BN / 2)) return VK_BAD_SHAPE;
-            return launch_wide<TC_SWIGLU>(mx, mw, out, M, 2 * N, K, error, stream, ex);
-        }
-        ex.group_rows = N;
-        if (!make_map(&mw, w, groups * N, K, K, TW_BN)) return VK_BAD_SHAPE;
-        if (mode == 0) return launch_wide<TC_SAME>(mx, mw, out, M, N, K, error, stream, ex);
-        return launch_wide<TC_F32>(mx, mw, out, M, N, K, error, stream, ex);
-    }
     if (gated) {
         ex.inter = N;
         ex.group_rows = 2 * N;
@@ -920,7 +928,7 @@ VK_API int vk_linear_tcgen05_grouped(const void* x, const void* w, void* out, in
         return launch_tc<128, TC_SWIGLU>(mx, mw, out, M, 2 * N, K, error, stream, ex);
     }
     ex.group_rows = N;
-    const int bn = N >= 2048 ? 128 : 64;
+    const int bn = N >= 1024 ? 128 : 64;           // the weights differ from tile to tile: wider tiles pay sooner than with one matrix
     if (!make_map(&mx, x, M, K, ldx, TC_BM) || !make_map(&mw, w, groups * N, K, K, bn)) return VK_BAD_SHAPE;
     if (bn == 128) {
         if (mode == 0) return launch_tc<128, TC_SAME>(mx, mw, out, M, N, K, error, stream, ex);

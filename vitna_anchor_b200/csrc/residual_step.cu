@@ -181,7 +181,7 @@ __global__ void __launch_bounds__(256) token_gate_kernel(const float* __restrict
     }
 }
 
-constexpr int TS_BLOCKS = 8, TS_THREADS = 256, TS_WARPS = TS_THREADS / 32;
+constexpr int TS_BLOCKS = 8, TS_THREADS = 512, TS_WARPS = TS_THREADS / 32;
 
 // Dot product of a row of T with float32 values in shared memory, the whole warp on one row.
 template <typename T>
@@ -191,7 +191,7 @@ __device__ __forceinline__ float ts_dot(const T* __restrict__ w, const float* s,
     return warp_sum(acc);
 }
 
-constexpr int TS_ROWS = 4;      // rows of the first product that a warp reads side by side
+constexpr int TS_ROWS = 2;      // rows of the first product that a warp reads side by side
 constexpr int TS_AHEAD = 8;     // pieces of the second product's rows on their way together
 
 template <typename T>
@@ -260,7 +260,7 @@ __global__ void __launch_bounds__(TS_THREADS) token_side_kernel(const StepArgs<T
             float acc[TS_ROWS];
 #pragma unroll
             for (int q = 0; q < TS_ROWS; q++) { w[q] = sd.gate + (size_t)min(r + q * STRIDE, dim - 1) * n; acc[q] = 0.0f; }
-#pragma unroll 2
+#pragma unroll 4
             for (int i = lane * V; i < n; i += 32 * V) {
                 float f[TS_ROWS][V];
 #pragma unroll
@@ -284,22 +284,26 @@ __global__ void __launch_bounds__(TS_THREADS) token_side_kernel(const StepArgs<T
     } else {
         for (int r = warp * TS_BLOCKS + rank; r < dim; r += STRIDE) give(r, ts_dot<T>(sd.gate + (size_t)r * n, xs, n, lane));
     }
+    // this block's rows of z; a row is dim / V pieces: several rows a warp where it is short.  The first pieces are asked for before the
+    // blocks meet.
+    int lanes = 1;
+    while (lanes < 32 && lanes * V < dim) lanes *= 2;
+    const int rows = 32 / lanes, sub = lane / lanes, in = lane - sub * lanes, step = TS_WARPS * rows, first = lo + warp * rows + sub;
+    uint4 piece[TS_AHEAD];
+    auto ask = [&](int r0, int i) {
+#pragma unroll
+        for (int q = 0; q < TS_AHEAD; q++) piece[q] = *reinterpret_cast<const uint4*>(sd.proj + (size_t)min(r0 + q * step, hi - 1) * dim + i);
+    };
+    if (vec_proj && first - sub < hi && in * V < dim) ask(first, in * V);
     cluster.sync();
-    // this block's rows of z
     float ss = 0.0f;
-    if (vec_proj) {                                     // a row is dim / V pieces: several rows a warp where it is short
-        int lanes = 1;
-        while (lanes < 32 && lanes * V < dim) lanes *= 2;
-        const int rows = 32 / lanes, sub = lane / lanes, in = lane - sub * lanes, step = TS_WARPS * rows;
-        for (int r0 = lo + warp * rows + sub; r0 - sub < hi; r0 += step * TS_AHEAD) {
+    if (vec_proj) {
+        for (int r0 = first; r0 - sub < hi; r0 += step * TS_AHEAD) {
             float acc[TS_AHEAD];
 #pragma unroll
             for (int q = 0; q < TS_AHEAD; q++) acc[q] = 0.0f;
             for (int i = in * V; i < dim; i += lanes * V) {
-                uint4 piece[TS_AHEAD];
-#pragma unroll
-                for (int q = 0; q < TS_AHEAD; q++)
-                    piece[q] = *reinterpret_cast<const uint4*>(sd.proj + (size_t)min(r0 + q * step, hi - 1) * dim + i);
+                if (r0 != first || i != in * V) ask(r0, i);
                 float gv[V];
 #pragma unroll
                 for (int e = 0; e < V; e += 4) *reinterpret_cast<float4*>(gv + e) = *reinterpret_cast<const float4*>(g + i + e);

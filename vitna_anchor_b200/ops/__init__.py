@@ -1962,6 +1962,21 @@ def token_gate(a: torch.Tensor, side: torch.Tensor, off: int, ids: torch.Tensor,
     return out
 
 
+def linear_token_gate(x: torch.Tensor, w: torch.Tensor, side: torch.Tensor, off: int, ids: torch.Tensor, a: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out [T, dim] = gelu_tanh(x @ w.T) * side[ids, off : off + dim].  In bfloat16 for more than a few rows the gelu and the factor are the epilogue of
+    the tcgen05 product; elsewhere the product leaves a (float32 [T, dim], scratch) and token_gate follows."""
+    T, W = x.shape
+    dim = w.shape[0]
+    if T > SKINNY_MAX_ROWS and x.dtype == w.dtype == torch.bfloat16 and tcgen05_takes(x, w) and out.data_ptr() % 16 == 0:
+        _req(w, "w", torch.bfloat16, 2); _req(out, "out", torch.bfloat16, 2); _req(side, "side", torch.bfloat16, 2); _req(ids, "ids", torch.int32, 1)
+        if w.shape[1] != W or out.shape != (T, dim) or ids.shape[0] < T or off < 0 or off + dim > side.shape[1]:
+            raise KernelError("linear_token_gate: shapes do not fit")
+        _check(lib().vk_linear_tcgen05_token(_p(x), _p(w), _p(out), T, dim, W, x.stride(0), _p(side), side.shape[1], off, _p(ids), side.shape[0],
+                                             _p(error_word()), _stream()), "linear_tcgen05_token")
+        return out
+    return token_gate(linear(x, w, a, LINEAR_F32), side, off, ids, out)
+
+
 def token_side_takes(dtype: torch.dtype, rows: int, n: int, dim: int) -> bool:
     """Whether residual_step and the per-layer input run as one kernel: few tokens (not in the exact 32-bit routing), a row that fits."""
     fn = lib().vk_token_side_smem

@@ -240,8 +240,8 @@ class ScaledResidualBlock(Block):
             ws = ctx.workspace
             xc = x if ctx.dtype == torch.float32 else ws.rows("scaled.xc", T, W, ctx.dtype)
             ops.residual_step(x, y, scale, out=None if xc is x else xc, eps=eps)
-            a = ops.linear(xc, side.gate, ws.rows("side.a", T, side.dim, torch.float32), ops.LINEAR_F32)
-            g = ops.token_gate(a, side.side, side.off, ctx.tokens, ws.rows("side.g", T, side.dim, ctx.dtype))
+            g = ops.linear_token_gate(xc, side.gate, side.side, side.off, ctx.tokens, ws.rows("side.a", T, side.dim, torch.float32),
+                                      ws.rows("side.g", T, side.dim, ctx.dtype))
             z = ops.linear(g, side.proj, ws.rows("side.z", T, W, torch.float32), ops.LINEAR_F32)
             ops.residual_step(x, z=z, z_norm=side.weight, mult=side.mult, **rest)
 
