@@ -45,7 +45,7 @@ class RotaryAttention(SplitMixer):
             raise ValueError("the projections' bias does not fit their rows")
         if rot_dims % 2 or rot_dims > dim or (rot_dims and (freq is None or freq.shape != (rot_dims // 2,))):
             raise ValueError("the rotation does not fit the heads")
-        if w_in.shape[0] % 4:                   # the product's rows end on 16 bytes whatever the number of gates
+        if gate and w_in.shape[0] % 4:          # the product's rows end on 16 bytes whatever the number of gates
             w_in = torch.cat([w_in, torch.zeros(4 - w_in.shape[0] % 4, hidden, dtype=w_in.dtype, device=w_in.device)], dim=0)
         super().__init__(w_in, w_out)
         self.hidden, self.H, self.G, self.dim, self.vdim, self.scale = hidden, H, G, dim, vdim, float(scale)
